@@ -3,7 +3,7 @@
 //
 // One CTA per SM.  A single producer thread walks this CTA's static slice of the weight matrix
 // and keeps a ring of shared-memory stages full with 1-D bulk async copies
-// (cp.async.bulk ... mbarrier::complete_tx, SASS UBLKCP); eight consumer warps pop tiles, do the
+// (cp.async.bulk ... mbarrier::complete_tx); eight consumer warps pop tiles, do the
 // int8 x int8 dot products with dp4a and reduce each row's per-block terms in the exact order of
 // Q8_0FloatTensor.dotQ8Activation (Q8_0FloatTensor.java:90-123).  The producer never waits for
 // anything but ring space: under programmatic dependent launch the NEXT matvec kernel is already
