@@ -13,7 +13,7 @@
 //   * k_delta_rule_reg  the recurrence S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with the state in registers: eight
 //                       lanes share a state column, the rows of a chunk run in sequence, columns in parallel over warps and CTAs;
 //   * k_delta_rule      the same for key sizes above 128: one thread per state column, the state tile in shared memory;
-//   * k_head_norm_gate  per-head RMS norm of the read-out, weight, SiLU gate.
+//   * k_head_norm_gate  per-head RMS norm of the read-out (optionally divided by a denominator per head first), weight, SiLU or sigmoid gate.
 // Rotation, scores, decays, gates, unit norms and the state are FP32 in both compute modes; fmaf is explicit because the
 // translation unit is compiled with -fmad=false.
 #pragma once
@@ -329,19 +329,30 @@ __global__ void __launch_bounds__(DR_THREADS) k_delta_rule_reg(const float *__re
     for (int i = 0; i < R; i++) Sg[(size_t)i * DR_THREADS] = Sr[i];
 }
 
-// One CTA per row, one warp per head: y = o / sqrt(mean(o^2) + eps) * w[d] * silu(gate[h][d]).
-__global__ void __launch_bounds__(256) k_head_norm_gate(const float *__restrict__ O, int ldo, const float *__restrict__ G, int ldg, const float *__restrict__ w, int heads, int dv,
-                                                        float eps, float *__restrict__ out32, bf16 *__restrict__ out16, int ldout) {
-    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int h = warp; h < heads; h += 8) {
+// One CTA per row, one warp per head: y = o / sqrt(mean(o^2) + eps) * w[h * w_stride + d] * gate(g[h][d]), gate = silu (sigmoid_gate: sigmoid).
+// w_stride: 0 = one weight of size dv for all heads, dv = a weight per head.  den (nullable, row stride ldo): o is O / den[h].
+struct HeadNormArgs {
+    const float *w;
+    int w_stride, sigmoid_gate;
+    const float *den;
+    int heads, dv;
+    float eps;
+};
+__global__ void __launch_bounds__(256) k_head_norm_gate(const float *__restrict__ O, int ldo, const float *__restrict__ G, int ldg, HeadNormArgs a, float *__restrict__ out32,
+                                                        bf16 *__restrict__ out16, int ldout) {
+    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, heads = a.heads, dv = a.dv;
+    const float eps = a.eps;
+    for (int h = blockIdx.y * 8 + warp; h < heads; h += 8 * gridDim.y) {
+        const float *w = a.w + (size_t)h * a.w_stride;
+        const float rden = a.den ? 1.0f / a.den[(size_t)r * ldo + h] : 1.0f;
         const float *o = O + (size_t)r * ldo + (size_t)h * dv, *g = G + (size_t)r * ldg + (size_t)h * dv;
         float ss = 0.0f;
-        for (int i = lane; i < dv; i += 32) ss = fmaf(o[i], o[i], ss);
+        for (int i = lane; i < dv; i += 32) { const float v = o[i] * rden; ss = fmaf(v, v, ss); }
         ss = warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+        const float inv = rden / sqrtf(ss / (float)dv + eps);
         for (int i = lane; i < dv; i += 32) {
             const float z = g[i];
-            const float y = o[i] * inv * w[i] * (z / (1.0f + expf(-z)));
+            const float y = o[i] * inv * w[i] * ((a.sigmoid_gate ? 1.0f : z) / (1.0f + expf(-z)));
             if (out32) out32[(size_t)r * ldout + (size_t)h * dv + i] = y;
             if (out16) out16[(size_t)r * ldout + (size_t)h * dv + i] = __float2bfloat16_rn(y);
         }

@@ -2,8 +2,9 @@
 // layered.cuh and sharing its projection and attention kernels:
 //   * k_block_norm_rows  the PARALLEL block's row kernel: x += mult * (a + sum of the feed-forward's per-slot results), then
 //                        TWO norms of the same x (layer norm with weight and bias, one pair per branch) in one pass; also the
-//                        embedding gather and the gathered final norm;
-//   * k_latent_prep      latent attention: RMS norm of the key/value latent, rotation of the shared key part and of every
+//                        embedding gather (optionally plus a hashed bigram row and a sinusoidal position vector) and the gathered
+//                        final norm;
+//   * k_latent_prep      latent attention: RMS norm of the key/value latent (and of the query latent), rotation of the shared key part and of every
 //                        head's rotated query part (table-driven: half-split or interleaved pairs, any blend of frequencies),
 //                        cache write [latent | rotated shared key part];
 //   * k_moe_route        router logits in FP32, sigmoid scores and selection of the `top` largest per row;
@@ -24,10 +25,15 @@ struct BlockNormArgs {
     const int *tokens;    // [n] (nullable: the step's own token)
     const StepState *st;
     float emb_scale;
+    const bf16 *bigram;   // (nullable) [buckets + 1][E], added to the embedding: row (prev * mul_prev + token * mul_cur) mod buckets, the last row at position 0
+    int bg_buckets, bg_prev, bg_cur;
+    int *tok_hist;        // (with bigram) token of every position: this launch's tokens are written, the one before its first row is read
+    const double *pos_freq; // (nullable) [(E + 1) / 2]: entry 2i += sin(pos * pos_freq[i]), entry 2i + 1 += cos(pos * pos_freq[i])
     const float *add_a;   // [n][E] (nullable): mixer output of the previous layer
     const float *add_b;   // [n * add_b_terms][E] (nullable): feed-forward results, row r owns entries r * terms .. r * terms + terms - 1
     const int *add_b_map; // (nullable) entry e lives in row add_b_map[e] of add_b (results left in expert-sorted order)
     int add_b_terms;
+    const float *add_b_wts; // (nullable) [n * add_b_terms]: weight of every entry
     float add_mult;       // x += add_mult * (a + sum b)
     float *trace;         // [n][E]: copy of x after the update (nullable)
     const float *w1, *b1; // first norm (nullable: no output); b nullable
@@ -42,44 +48,93 @@ struct BlockNormArgs {
     int E;
 };
 
-__global__ void __launch_bounds__(LY_NORM_THREADS) k_block_norm_rows(BlockNormArgs a) {
+#define LY_BLOCK_TERMS 64 // feed-forward results of a row whose places and weights are kept in shared memory (more: read where they are)
+// sin / cos of pos * f with the angle and its reduction to [-pi, pi] in double precision, the function itself in FP32
+__device__ __forceinline__ float sinusoid_entry(int pos, double f, bool cosine) {
+    const double a = (double)pos * f;
+    const float r = (float)fma(-rint(a * 0.15915494309189533577), 6.283185307179586476925, a);
+    return cosine ? cosf(r) : sinf(r);
+}
+// One CTA of NTH threads per row (a single wide row takes more threads: more of its loads are in flight)
+template <int NTH>
+__global__ void __launch_bounds__(NTH) k_block_norm_rows(BlockNormArgs a) {
     extern __shared__ __align__(16) float row[];
     __shared__ float red[32];
+    __shared__ size_t s_row[LY_BLOCK_TERMS]; // offset of a feed-forward result row
+    __shared__ float s_wt[LY_BLOCK_TERMS];
     const int r = blockIdx.x, tid = threadIdx.x, E = a.E;
+    const bool terms = a.add_b && a.add_b_terms <= LY_BLOCK_TERMS;
+    if (terms) {
+        if (tid < a.add_b_terms) {
+            const size_t e = (size_t)r * a.add_b_terms + tid;
+            s_row[tid] = (a.add_b_map ? (size_t)a.add_b_map[e] : e) * E;
+            s_wt[tid] = a.add_b_wts ? a.add_b_wts[e] : 1.0f;
+        }
+        __syncthreads();
+    }
     const size_t src = (size_t)(a.gather ? a.gather[r] : r) * E, dst = (size_t)r * E;
     if (a.emb) {
         const int token = a.tokens ? a.tokens[r] : a.st->token;
         const bf16 *e = a.emb + (size_t)token * E;
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] = __bfloat162float(e[i]) * a.emb_scale;
+        const int pos = (a.bigram || a.pos_freq) ? a.st->pos + r : 0;
+        const bf16 *bg = nullptr;
+        if (a.bigram) {
+            long long b = a.bg_buckets;
+            if (pos > 0) {
+                const long long prev = r > 0 ? a.tokens[r - 1] : a.tok_hist[pos - 1];
+                b = (prev * a.bg_prev + (long long)token * a.bg_cur) % a.bg_buckets;
+            }
+            bg = a.bigram + (size_t)b * E;
+            if (tid == 0) a.tok_hist[pos] = token;
+        }
+        for (int i = tid; i < E; i += NTH) {
+            float v = __bfloat162float(e[i]) * a.emb_scale;
+            if (bg) v += __bfloat162float(bg[i]);
+            if (a.pos_freq) v += sinusoid_entry(pos, a.pos_freq[i >> 1], i & 1);
+            row[i] = v;
+        }
     } else {
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] = a.x[src + i];
+        for (int i = tid; i < E; i += NTH) row[i] = a.x[src + i];
     }
-    if (a.add_a || a.add_b) {
-        for (int i = tid; i < E; i += LY_NORM_THREADS) {
+    if (terms) {
+        for (int i = tid; i < E; i += NTH) {
+            float s = a.add_a ? a.add_a[src + i] : 0.0f;
+            for (int k0 = 0; k0 < a.add_b_terms; k0 += 4) { // the loads of four results are issued before the first is used
+                float v[4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) v[u] = k0 + u < a.add_b_terms ? __ldg(a.add_b + s_row[k0 + u] + i) : 0.0f;
+#pragma unroll
+                for (int u = 0; u < 4; u++) if (k0 + u < a.add_b_terms) s = fmaf(s_wt[k0 + u], v[u], s);
+            }
+            row[i] = fmaf(a.add_mult, s, row[i]);
+        }
+    } else if (a.add_a || a.add_b) {
+        for (int i = tid; i < E; i += NTH) {
             float s = a.add_a ? a.add_a[src + i] : 0.0f;
             for (int k = 0; k < a.add_b_terms; k++) {
                 const size_t e = (size_t)r * a.add_b_terms + k;
-                s += a.add_b[(a.add_b_map ? (size_t)a.add_b_map[e] : e) * E + i];
+                const float v = a.add_b[(a.add_b_map ? (size_t)a.add_b_map[e] : e) * E + i];
+                s = a.add_b_wts ? fmaf(a.add_b_wts[e], v, s) : s + v;
             }
             row[i] = fmaf(a.add_mult, s, row[i]);
         }
     }
     if (!a.gather && (a.emb || a.add_a || a.add_b))
-        for (int i = tid; i < E; i += LY_NORM_THREADS) a.x[src + i] = row[i];
+        for (int i = tid; i < E; i += NTH) a.x[src + i] = row[i];
     if (a.trace)
-        for (int i = tid; i < E; i += LY_NORM_THREADS) a.trace[src + i] = row[i];
+        for (int i = tid; i < E; i += NTH) a.trace[src + i] = row[i];
     if (!a.w1 && !a.w2) return;
     float mean = 0.0f;
     if (!a.rms) {
         float s = 0.0f;
-        for (int i = tid; i < E; i += LY_NORM_THREADS) s += row[i];
+        for (int i = tid; i < E; i += NTH) s += row[i];
         mean = block_sum(s, red) / (float)E;
     }
     float ss = 0.0f;
-    for (int i = tid; i < E; i += LY_NORM_THREADS) { const float d = row[i] - mean; ss = fmaf(d, d, ss); }
+    for (int i = tid; i < E; i += NTH) { const float d = row[i] - mean; ss = fmaf(d, d, ss); }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
-    for (int i = tid; i < E; i += LY_NORM_THREADS) {
+    for (int i = tid; i < E; i += NTH) {
         const float u = (row[i] - mean) * inv;
         if (a.w1) {
             const float v = fmaf(u, a.w1[i], a.b1 ? a.b1[i] : 0.0f);
@@ -106,6 +161,12 @@ struct LatentArgs {
     int rope_dims;       // the first rope_dims entries of a rotated part turn, the rest pass unchanged
     int rope_layout;     // 0: pair (i, i + rope_dims / 2);  1: pair (2i, 2i + 1)
     float eps;
+    // queries through a latent of their own: q_off names the query latent's columns (q_rank of them) instead of the queries', which a
+    // later product makes (no rotated part then); grid (rows, 2), the second CTA of a row norms the query latent into cq32 / cq16 [n][q_rank]
+    int q_rank;
+    const float *qnorm;  // [q_rank]
+    float *cq32;
+    bf16 *cq16;
 };
 
 __device__ __forceinline__ void rope_pair_index(int i, int dims, int layout, int &u, int &v) {
@@ -124,6 +185,19 @@ __global__ void __launch_bounds__(256) k_latent_prep(float *__restrict__ P, int 
     const int pos = st->pos + r, half = a.rope_dims / 2, kw = a.rank + a.dr;
     float *p = P + (size_t)r * ldp;
     const float *cs = a.cs + (size_t)pos * half * 2;
+    if (blockIdx.y == 1) {
+        const float *c = p + a.q_off;
+        float ss = 0.0f;
+        for (int i = tid; i < a.q_rank; i += 256) ss = fmaf(c[i], c[i], ss);
+        ss = block_sum(ss, red);
+        const float inv = 1.0f / sqrtf(ss / (float)a.q_rank + a.eps);
+        for (int i = tid; i < a.q_rank; i += 256) {
+            const float v = c[i] * inv * a.qnorm[i];
+            if (a.cq32) a.cq32[(size_t)r * a.q_rank + i] = v;
+            if (a.cq16) a.cq16[(size_t)r * a.q_rank + i] = __float2bfloat16_rn(v);
+        }
+        return;
+    }
     if (a.kv_off >= 0) {
         const float *c = p + a.kv_off, *kr = c + a.rank;
         float ss = 0.0f;
@@ -146,6 +220,7 @@ __global__ void __launch_bounds__(256) k_latent_prep(float *__restrict__ P, int 
             for (int i = tid; i < kw; i += 256) row16[i] = __float2bfloat16_rn(row[i]);
         }
     }
+    if (a.q_rank > 0) return;
     const int hw = a.dk + a.dr;
     float *q = Q + (size_t)r * a.heads * kw;
     for (int e = tid; e < a.heads * half; e += 256) {
@@ -176,17 +251,23 @@ __global__ void __launch_bounds__(256) k_latent_prep(float *__restrict__ P, int 
 // How the router's logits become expert ids and weights.  softmax == 0: scores sigmoid(z), the `top` largest, weight = score.
 // softmax == 1: scores s = softmax(z) over all router outputs, the `top` largest of s + correction are chosen, weight =
 // s / (sum of the chosen s + 1e-20) * scale.  Router outputs n_real .. are identity experts: they all get the id n_real.
+// softmax == 2: the `top` largest of z + bias, weights = softmax over those chosen values.
 struct RouteMode {
     int softmax;
     const float *correction; // [experts] (softmax mode)
     int n_real;              // experts with weights (<= experts)
     float scale;
+    const float *bias;       // [experts] (mode 2)
 };
 
 // One warp: z [experts] logits in shared memory (overwritten), sbuf [experts] scratch; ids / wts [top] in order of falling choice
 // score (the lowest index wins a tie).
 __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts, int top, const RouteMode &m, int *ids, float *wts, int lane) {
-    if (m.softmax) {
+    if (m.softmax == 2) {
+        for (int e = lane; e < experts; e += 32) z[e] += m.bias[e];
+        __syncwarp();
+    }
+    if (m.softmax == 1) {
         float mx = -INFINITY;
         for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
 #pragma unroll
@@ -197,7 +278,7 @@ __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts,
         for (int e = lane; e < experts; e += 32) { const float sc = sbuf[e] / sum; sbuf[e] = sc; z[e] = sc + m.correction[e]; }
         __syncwarp();
     }
-    float tot = 0.0f;
+    float tot = 0.0f, z_top = 0.0f;
     for (int k = 0; k < top; k++) {
         float best = -INFINITY;
         int bi = experts;
@@ -212,15 +293,18 @@ __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts,
         if (lane == 0) {
             const int id = bi < experts ? bi : 0;
             ids[k] = id < m.n_real ? id : m.n_real;
-            const float w = m.softmax ? (bi < experts ? sbuf[bi] : 0.0f) : 1.0f / (1.0f + expf(-best));
+            if (k == 0) z_top = best;
+            const float w = m.softmax == 2 ? expf(best - z_top) : m.softmax ? (bi < experts ? sbuf[bi] : 0.0f) : 1.0f / (1.0f + expf(-best));
             wts[k] = w;
             tot += w;
             if (bi < experts) z[bi] = -INFINITY; // taken
         }
         __syncwarp();
     }
-    if (m.softmax && lane == 0)
+    if (m.softmax == 1 && lane == 0)
         for (int k = 0; k < top; k++) wts[k] = wts[k] / (tot + 1e-20f) * m.scale;
+    if (m.softmax == 2 && lane == 0)
+        for (int k = 0; k < top; k++) wts[k] /= tot;
 }
 
 // Router: logits z_e = <Wr[e], x> accumulated in FP32 (x FP32 or its BF16 rounding, Wr BF16), then route_select; ids / wts

@@ -26,7 +26,7 @@ namespace ly {
 typedef __nv_bfloat16 bf16;
 
 enum { EPI_STORE = 0, EPI_GATED = 1, EPI_ACT = 2 }; // C = A W^T (+ bias)  |  H = act(A Wg^T) * (A Wu^T), W = [Wg; Wu] stacked by rows  |  H = act(A W^T (+ bias))
-enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_RELU = 2, ACT_GELU_ERF = 3 };
+enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_RELU = 2, ACT_GELU_ERF = 3, ACT_RELU2 = 4 };
 
 __device__ __forceinline__ float bf_lo(unsigned v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf_hi(unsigned v) { return __uint_as_float(v & 0xffff0000u); }
@@ -34,6 +34,7 @@ __device__ __forceinline__ float bf_hi(unsigned v) { return __uint_as_float(v & 
 __device__ __forceinline__ float act_apply(int act, float z) {
     if (act == ACT_SILU) return z / (1.0f + expf(-z));
     if (act == ACT_RELU) return fmaxf(z, 0.0f);
+    if (act == ACT_RELU2) { const float r = fmaxf(z, 0.0f); return r * r; }
     if (act == ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); // the exact GELU: z * Phi(z)
     // tanh form of GELU: 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
     const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);

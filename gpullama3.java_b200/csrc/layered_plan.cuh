@@ -21,12 +21,13 @@
 // experts reading two norms of the same residual row).  Sandwich and pre-norm layers choose their mixer per layer: windowed
 // attention (optionally with rotation, values taken from the keys, head temperatures and head-mixed scores: k_rope_mix_prep
 // replaces k_qk_prep) or the gated delta rule (k_delta_prep -> k_delta_rule -> k_head_norm_gate), whose recurrent state and
-// convolution inputs live per RUN next to the rings.
+// convolution inputs live per RUN next to the rings.  Two further block kinds: outnorm_plan.cuh, layernorm_plan.cuh.
 #pragma once
 #include "layered.cuh"
 #include "latent.cuh"
 #include "delta.cuh"
 #include "recurrent.cuh"
+#include "mlstm.cuh"
 
 struct LyLayer {
     b200_layer_spec s{};
@@ -43,6 +44,12 @@ struct LyLayer {
     ly::bf16 *w_uk = nullptr;                   // [heads * key_dim][kv_rank] as stored: the BF16 prefill that expands keys per head reads it
     bool expand = false;                        // BF16 prefill through expanded keys / values and the tensor-core attention kernel
     float *cnorm = nullptr;
+    ly::bf16 *w_uq = nullptr;                   // [heads * key_dim][q_rank]: queries out of the normed query latent (qnorm)
+    CUtensorMap m_uq, m_cq, m_qf_c;
+    bool tc_uq = false;
+    float *router_b = nullptr;
+    // matrix memory (B200_MIXER_MLSTM): gate biases; the fused projection is q | k | v | g | i | f, onorm the read-out weight [heads * value_dim]
+    float *i_bias = nullptr, *f_bias = nullptr;
     const float *rope = nullptr;                // [context][rope_dims / 2][2], shared between layers with the same rotation
     // parallel block: biases of the two layer norms; mixture of experts: router [experts][width], w_gu = [experts][2 ff][width],
     // w_down = [experts][width][ff]
@@ -114,6 +121,9 @@ struct Layered {
     float *final_norm_b = nullptr;
     float *A2_32 = nullptr, *Q = nullptr, *LAT32 = nullptr, *YS = nullptr, *moe_wts = nullptr, *ZR = nullptr;
     ly::bf16 *A2_16 = nullptr, *QU16 = nullptr, *LAT16 = nullptr;
+    float *CQ32 = nullptr, *QF = nullptr;      // normed query latents, queries made from them
+    ly::bf16 *CQ16 = nullptr;
+    int maxRq = 0;
     float *KXF = nullptr, *VXF = nullptr;      // FP32 results of the tcgen05 expansions, rows padded to whole 128-row tiles
     ly::bf16 *KX16 = nullptr, *VX16 = nullptr; // keys / values of one layer expanded per head for a prefill chunk: [context][heads * size]
     int maxKX = 0, maxVX = 0, pf_pos = 0;      // pf_pos: first position of the chunk being enqueued
@@ -138,6 +148,10 @@ struct Layered {
     ly::bf16 *U16 = nullptr;
     int max_att_heads = 1;
     CUtensorMap m_sh_c;
+    // LAYERNORM block: bigram table, token of every position, frequencies of the sinusoidal position vector
+    ly::bf16 *bigram = nullptr;
+    int *tok_hist = nullptr;
+    double *pos_freq = nullptr;
 };
 
 // What ly_project needs to take the tcgen05 route: operand and result descriptors (nullptr = CUDA-core / mma.sync kernels).
@@ -292,6 +306,7 @@ static int ly_project(b200_plan *p, bool decode, int n, const float *a32, const 
 
 #include "latent_plan.cuh"
 #include "outnorm_plan.cuh"
+#include "layernorm_plan.cuh"
 
 // Enqueue the forward of n rows on p->stream.  decode: the single-token step (row 0, position and token from *st).
 // with_head (decode only): final norm + classifier into p->logits.  Prefill leaves the finished residual rows in X.
@@ -299,6 +314,7 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
     Layered &Y = *p->ly;
     if (Y.c.block == B200_BLOCK_PARALLEL) return ly_enqueue_parallel(p, decode, n, st, tokens, with_head, trace, launches);
     if (Y.c.block == B200_BLOCK_OUTNORM) return ly_enqueue_outnorm(p, decode, n, st, tokens, with_head, trace, launches);
+    if (Y.c.block == B200_BLOCK_LAYERNORM) return ly_enqueue_layernorm(p, decode, n, st, tokens, with_head, trace, launches);
     const int E = Y.c.width;
     const bool h16 = !decode && !Y.f32; // prefill in BF16 mode rounds GEMM operands to BF16
     int nl = 0, rc;
@@ -351,8 +367,9 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
                               (const float *)Y.DLT, Y.maxD, da, R.S, n, Y.DO, Y.maxDO, st);
             }
             if (rc) return rc;
-            if ((rc = launch_k(p, false, ly::k_head_norm_gate, dim3(n), dim3(256), (size_t)0, (const float *)Y.DO, Y.maxDO, (const float *)(Y.PROJ + L.dC + 2 * L.s.heads), Y.maxP,
-                               (const float *)L.onorm, L.s.heads, L.s.value_dim, Y.c.norm_eps, h16 ? (float *)nullptr : Y.ATT32, h16 ? Y.ATT16 : (ly::bf16 *)nullptr, L.gd))) return rc;
+            const ly::HeadNormArgs ha{L.onorm, 0, 0, nullptr, L.s.heads, L.s.value_dim, Y.c.norm_eps};
+            if ((rc = launch_k(p, false, ly::k_head_norm_gate, dim3(n), dim3(256), (size_t)0, (const float *)Y.DO, Y.maxDO, (const float *)(Y.PROJ + L.dC + 2 * L.s.heads), Y.maxP, ha,
+                               h16 ? (float *)nullptr : Y.ATT32, h16 ? Y.ATT16 : (ly::bf16 *)nullptr, L.gd))) return rc;
             nl += 3;
         } else {
         const ly::WindowAttn wa = ly_attn_args(Y, L);
@@ -470,10 +487,20 @@ static int ly_tc_init(b200_plan *p) {
         for (LyLayer &L : Y.layers) {
             if (L.s.ff_kind != B200_FF_MOE || L.s.ff_dim % 64) continue;
             const uint64_t F = L.s.ff_dim, X = L.s.ff_experts;
+            if (L.s.moe_plain) { // one matrix in front of the activation, tiles of 128 of its rows
+                L.tc_moe = F % 128 == 0 && pg::make_map(&L.m_moe_up, L.w_gu, X * F, E, pg::BN) == 0 && pg::make_map(&L.m_moe_down, L.w_down, X * E, F, pg::BN) == 0 &&
+                           pg::make_map(&L.m_moe_h, Y.HS16, (uint64_t)Y.max_tiles128 * 128, F, pg::BM) == 0;
+                continue;
+            }
             L.tc_moe = pg::make_map(&L.m_moe_gate, L.w_gu, X * 2 * F, E, pg::BN / 2) == 0 && pg::make_map(&L.m_moe_up, L.w_gu + F * E, X * 2 * F - F, E, pg::BN / 2) == 0 &&
                        pg::make_map(&L.m_moe_down, L.w_down, X * E, F, pg::BN) == 0 && pg::make_map(&L.m_moe_h, Y.HS16, (uint64_t)Y.max_tiles128 * 128, F, pg::BM) == 0;
         }
     if (Y.outnorm) ly_outnorm_tc_init(p);
+    for (LyLayer &L : Y.layers) { // queries out of a query latent
+        const int N = L.s.heads * L.s.key_dim, Rq = L.s.q_rank;
+        if (L.s.mixer == B200_MIXER_LATENT_ATTENTION && Rq > 0)
+            L.tc_uq = fits(N, Rq) && pg::make_map(&L.m_uq, L.w_uq, N, Rq, 128) == 0 && pg::make_map(&L.m_cq, Y.CQ16, rows, Rq, pg::BM) == 0 && pg::make_map_c(&L.m_qf_c, Y.QF, rows, N) == 0;
+    }
     Y.tc_head = fits(V, E) && pg::make_map(&Y.m_head, Y.head, V, E, 128) == 0 && pg::make_map_c(&Y.m_log_c, Y.LOG, 256, V) == 0;
     Y.tc = true;
     return B200_OK;
@@ -485,8 +512,8 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     Layered &Y = *Yp;
     Y.c = *cfg;
     const b200_layered_config &c = Y.c;
-    if (c.arch != B200_ARCH_PIBIDRA && c.arch != B200_ARCH_LATUSUN && c.arch != B200_ARCH_LEROSUN && c.arch != B200_ARCH_DINUZEN) return fail(p, B200_ERR_UNSUPPORTED, "unknown layered arch %d", c.arch);
-    if (c.block != B200_BLOCK_SANDWICH && c.block != B200_BLOCK_PARALLEL && c.block != B200_BLOCK_PRENORM && c.block != B200_BLOCK_OUTNORM) return fail(p, B200_ERR_BAD_ARG, "unknown block kind %d", c.block);
+    if (c.arch != B200_ARCH_PIBIDRA && c.arch != B200_ARCH_LATUSUN && c.arch != B200_ARCH_LEROSUN && c.arch != B200_ARCH_DINUZEN && c.arch != B200_ARCH_KEGASUN) return fail(p, B200_ERR_UNSUPPORTED, "unknown layered arch %d", c.arch);
+    if (c.block != B200_BLOCK_SANDWICH && c.block != B200_BLOCK_PARALLEL && c.block != B200_BLOCK_PRENORM && c.block != B200_BLOCK_OUTNORM && c.block != B200_BLOCK_LAYERNORM) return fail(p, B200_ERR_BAD_ARG, "unknown block kind %d", c.block);
     Y.outnorm = c.block == B200_BLOCK_OUTNORM;
     const bool outn = Y.outnorm;
     if (outn) {
@@ -496,7 +523,9 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     }
     Y.prenorm = c.block == B200_BLOCK_PRENORM;
     Y.w_off = Y.prenorm ? 0.0f : 1.0f;
-    const bool par = c.block == B200_BLOCK_PARALLEL;
+    const bool par = c.block == B200_BLOCK_PARALLEL, lnb = c.block == B200_BLOCK_LAYERNORM;
+    if (lnb && c.loop_times >= 0 && c.loop_stop > c.loop_start) return fail(p, B200_ERR_UNSUPPORTED, "layer-norm blocks do not loop");
+    if (lnb && (c.bigram_buckets < 0 || (c.sinusoid && !(c.sinusoid_base > 0.0f)))) return fail(p, B200_ERR_BAD_ARG, "%d bigram buckets, sinusoid base %g", c.bigram_buckets, (double)c.sinusoid_base);
     if (par && Y.has_loop && c.loop_stop > c.loop_start) return fail(p, B200_ERR_UNSUPPORTED, "parallel blocks do not loop");
     if (c.width <= 0 || c.vocab_size <= 0 || c.n_layers <= 0 || c.context_length <= 0) return fail(p, B200_ERR_BAD_ARG, "width, vocabulary, layers and context must be positive");
     if (c.compute != B200_COMPUTE_BF16 && c.compute != B200_COMPUTE_F32) return fail(p, B200_ERR_BAD_ARG, "compute must be B200_COMPUTE_BF16 or B200_COMPUTE_F32");
@@ -532,12 +561,18 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             if ((rc = ly_outnorm_sizes(p, l, L, specs))) return rc;
             continue;
         }
+        if (lnb) {
+            if ((rc = ly_layernorm_sizes(p, l, L, specs))) return rc;
+            continue;
+        }
         if (par) {
             // parallel block: latent attention and a mixture of experts (or no feed-forward)
             if (s.mixer != B200_MIXER_LATENT_ATTENTION) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: mixer %d in a parallel block", l, s.mixer);
             L.s.window = c.context_length; // causal over the whole sequence
             if ((rc = ly_latent_sizes(p, l, L, c.n_layers, specs))) return rc;
             if (s.ff_kind != B200_FF_NONE && s.ff_kind != B200_FF_MOE) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d in a parallel block", l, s.ff_kind);
+            if (s.q_rank || s.sink || s.gate > 1 || s.moe_plain || s.moe_router != B200_MOE_SIGMOID_INPUT)
+                return fail(p, B200_ERR_UNSUPPORTED, "layer %d: query latents, sinks, per-head gates, plain experts and softmax routers are not combined with the parallel block", l);
             if (s.ff_kind == B200_FF_MOE) {
                 if (s.ff_dim <= 0 || s.ff_experts <= 0 || (size_t)4 * (E + s.ff_experts) * 4 > (size_t)Y.smem_max || s.ff_top <= 0 || s.ff_top > s.ff_experts || (s.ff_act != B200_ACT_GELU_TANH && s.ff_act != B200_ACT_SILU))
                     return fail(p, B200_ERR_BAD_ARG, "layer %d: %d experts of width %d, %d chosen, activation %d", l, s.ff_experts, s.ff_dim, s.ff_top, s.ff_act);
@@ -545,13 +580,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
                 if (s.ff_top > Y.maxTop) Y.maxTop = s.ff_top;
                 if (s.ff_experts > Y.maxExperts) Y.maxExperts = s.ff_experts;
             }
-            if (L.P > Y.maxP) Y.maxP = L.P;
-            if (L.gd > Y.maxO) Y.maxO = L.gd;
-            if (L.qw > Y.maxQ) Y.maxQ = L.qw;
-            if (L.lw > Y.maxL) Y.maxL = L.lw;
-            if (s.heads * s.key_dim > Y.maxQU) Y.maxQU = s.heads * s.key_dim;
-            if (s.kv_rank > Y.max_att_dv) Y.max_att_dv = s.kv_rank;
-            if (L.s.window > Y.max_window) Y.max_window = L.s.window;
+            ly_latent_buffers(Y, L);
             continue;
         }
         if (s.mixer != B200_MIXER_WINDOW_ATTENTION && s.mixer != B200_MIXER_GATED_DELTA) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: mixer %d", l, s.mixer);
@@ -605,6 +634,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         int maxK = E > Y.maxO ? E : Y.maxO;
         if (Y.maxF > maxK) maxK = Y.maxF;
         for (const LyLayer &L : Y.layers) if (L.s.kv_rank > maxK) maxK = L.s.kv_rank; // reduction width of the per-head value expansion
+        if (Y.maxRq > maxK) maxK = Y.maxRq;
         size_t need = (size_t)maxK * 4;
         if (outn && (size_t)2 * E * 4 > need) need = (size_t)2 * E * 4; // the row kernel holds the row and the sublayer's output
         for (const LyLayer &L : Y.layers) if (ly_att_smem(L.s, 0) > need) need = ly_att_smem(L.s, 0);
@@ -612,7 +642,8 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         static bool attrs = false; // per function and process-wide, like plan.cu's set_smem_attrs
         if (!attrs) {
             CK(set_max_dyn(ly::k_norm_rows, Y.smem_max));
-            CK(set_max_dyn(ly::k_block_norm_rows, Y.smem_max));
+            CK(set_max_dyn(ly::k_block_norm_rows<LY_NORM_THREADS>, Y.smem_max));
+            CK(set_max_dyn(ly::k_block_norm_rows<1024>, Y.smem_max));
             CK(set_max_dyn(ly::k_moe_route<float>, Y.smem_max));
             CK(set_max_dyn(ly::k_moe_route<ly::bf16>, Y.smem_max));
             CK(set_max_dyn(ly::k_matvec_bf16<ly::EPI_STORE>, Y.smem_max));
@@ -636,11 +667,12 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     }
     // Latent attention, BF16 prefill: layers whose per-head key size (unrotated + rotated) and value size are an instance of the
     // tensor-core attention kernel expand keys and values per head for the chunk and run it; all others attend in the folded form
-    if (par && !Y.f32 && Y.att_mma && Y.cap > 1 && Y.maxP % 4 == 0)
+    if ((par || lnb) && !Y.f32 && Y.att_mma && Y.cap > 1 && Y.maxP % 4 == 0)
         for (LyLayer &L : Y.layers) {
+            if (L.s.mixer != B200_MIXER_LATENT_ATTENTION) continue;
             const int DK = L.s.key_dim + L.s.rot_dim;
             const int kind = ly_mma_kind(DK, L.s.value_dim);
-            L.expand = kind && ly_mma_smem(kind, L.s.window) <= (size_t)Y.smem_max && (!L.s.gate || L.g_off % 2 == 0) && L.s.key_dim % 8 == 0;
+            L.expand = kind && ly_mma_smem(kind, L.s.window) <= (size_t)Y.smem_max && (L.s.gate != 1 || L.g_off % 2 == 0) && L.s.key_dim % 8 == 0;
             if (L.expand) {
                 if (L.s.heads * DK > Y.maxKX) Y.maxKX = L.s.heads * DK;
                 if (L.gd > Y.maxVX) Y.maxVX = L.gd;
@@ -671,7 +703,8 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     if ((rc = ly_mat(p, tensors, nt, "embed", c.vocab_size, E, Y.emb, 0))) return rc;
     if ((rc = dalloc(p, &Y.head, (size_t)c.vocab_size * E * 2))) return rc;
     if ((rc = ly_mat(p, tensors, nt, "head", c.vocab_size, E, Y.head, 0))) return rc;
-    if (outn) {
+    if (lnb && (rc = ly_layernorm_embedding(p, tensors, nt))) return rc;
+    if (outn || lnb) {
         if ((rc = ly_vec_f32(p, tensors, nt, "final.norm", E, &Y.final_norm))) return rc;
     } else if (Y.prenorm) {
         if ((rc = ly_scalar_vec(p, tensors, nt, "final.norm", E, &Y.final_norm))) return rc;
@@ -690,6 +723,10 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         }
         if (outn) {
             if ((rc = ly_outnorm_upload(p, l, L, tensors, nt))) return rc;
+            continue;
+        }
+        if (lnb) {
+            if ((rc = ly_layernorm_upload(p, l, L, tensors, nt))) return rc;
             continue;
         }
         if (Y.prenorm) {
@@ -802,6 +839,12 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             }
             continue;
         }
+        if (L.s.mixer == B200_MIXER_MLSTM) { // the run's matrix memory, normaliser and running maximum
+            R.s_floats = ly::mlstm_state_floats(L.s.heads, L.s.key_dim, L.s.value_dim);
+            if ((rc = dalloc(p, &R.S, R.s_floats * 4))) return rc;
+            CK(cudaMemset(R.S, 0, R.s_floats * 4));
+            continue;
+        }
         if (L.s.mixer == B200_MIXER_GATED_DELTA) {
             // the run's recurrent state and its ring of convolution inputs (position j in slot j % cring)
             const size_t sb = ly::delta_state_floats(L.s.heads, L.s.key_dim, L.s.value_dim) * 4, cb = (size_t)Y.cring * L.dC * 4;
@@ -834,13 +877,14 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     const size_t slots = Y.maxTop > 0 ? (size_t)Y.maxTop : 1; // feed-forward rows per token (a mixture of experts: one per chosen expert)
     if ((rc = dalloc(p, &Y.X, cap * E * 4))) return rc;
     if (Y.has_loop && !Y.prenorm && (rc = dalloc(p, &Y.X0, cap * E * 4))) return rc;
-    if (!par && Y.maxQ > 0 && (rc = dalloc(p, &Y.Q, cap * Y.maxQ * 4))) return rc;
+    if (!par && !lnb && Y.maxQ > 0 && (rc = dalloc(p, &Y.Q, cap * Y.maxQ * 4))) return rc;
     if (outn) {
         if (Y.c.depth_average && (rc = dalloc(p, &Y.STASH, (size_t)(c.n_layers + 1) * Y.cap * E * 4))) return rc;
         if (Y.maxTop > 0 && ((rc = dalloc(p, &Y.SH, cap * E * 4)) || (rc = dalloc(p, &Y.SGL, cap * 4)))) return rc;
         if (!Y.f32 && Y.maxD > 0 && (rc = dalloc(p, &Y.U16, cap * Y.maxD * 2))) return rc;
         if (Y.maxDO > 0 && !Y.DO && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
     }
+    if (lnb && Y.maxDO > 0 && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
     if (Y.maxD > 0 && ((rc = dalloc(p, &Y.DLT, cap * Y.maxD * 4)) || (rc = dalloc(p, &Y.DO, cap * (Y.maxDO > 0 ? Y.maxDO : 1) * 4)))) return rc;
     if ((rc = dalloc(p, &Y.Y, cap * E * 4))) return rc;
     if ((rc = dalloc(p, &Y.PROJ, cap * Y.maxP * 4))) return rc;
@@ -852,7 +896,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         if ((rc = dalloc(p, &Y.ATT16, cap * Y.maxO * 2))) return rc;
         if ((rc = dalloc(p, &Y.H16, cap * slots * maxF * 2))) return rc;
     }
-    if (par || outn) {
+    if (par || outn || lnb) {
         if (Y.maxKX > 0) {
             if ((rc = dalloc(p, &Y.KX16, (size_t)Y.ring * Y.maxKX * 2))) return rc;
             if ((rc = dalloc(p, &Y.VX16, (size_t)Y.ring * Y.maxVX * 2))) return rc;
@@ -861,10 +905,16 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             if ((rc = dalloc(p, &Y.VXF, rowsX * Y.maxVX * 4))) return rc;
         }
         if (par && (rc = dalloc(p, &Y.A2_32, rows32 * E * 4))) return rc;
-        if (par && (rc = dalloc(p, &Y.Q, cap * Y.maxQ * 4))) return rc;
-        if (par && (rc = dalloc(p, &Y.LAT32, rows32 * Y.maxL * 4))) return rc;
-        if (par && !Y.f32) {
-            if ((rc = dalloc(p, &Y.A2_16, cap * E * 2))) return rc;
+        const bool lat = par || (lnb && Y.maxL > 0);
+        if (lat && (rc = dalloc(p, &Y.Q, cap * Y.maxQ * 4))) return rc;
+        if (lat && (rc = dalloc(p, &Y.LAT32, rows32 * Y.maxL * 4))) return rc;
+        if (Y.maxRq > 0) {
+            if ((rc = dalloc(p, &Y.CQ32, rows32 * Y.maxRq * 4))) return rc;
+            if ((rc = dalloc(p, &Y.QF, cap * Y.maxQU * 4))) return rc;
+            if (!Y.f32 && (rc = dalloc(p, &Y.CQ16, cap * Y.maxRq * 2))) return rc;
+        }
+        if (par && !Y.f32 && (rc = dalloc(p, &Y.A2_16, cap * E * 2))) return rc;
+        if (lat && !Y.f32) {
             if ((rc = dalloc(p, &Y.QU16, cap * Y.maxQU * 2))) return rc;
             if ((rc = dalloc(p, &Y.LAT16, cap * Y.maxL * 2))) return rc;
         }
@@ -968,11 +1018,11 @@ static int ly_batch(b200_plan *p, const int32_t *tokens, int n, int start_pos, c
             a.w_out = Y.final_norm; a.gather = Y.rows; a.st = Y.st_pf;
             a.out32 = Y.f32 ? Y.A32 : nullptr; a.out16 = Y.f32 ? nullptr : Y.A16;
             if ((rc = launch_k(p, false, ly::k_outnorm_rows<LY_NORM_THREADS>, dim3(m), dim3(LY_NORM_THREADS), (size_t)2 * E * 4, a))) return rc;
-        } else if (Y.c.block == B200_BLOCK_PARALLEL) {
+        } else if (Y.c.block == B200_BLOCK_PARALLEL || Y.c.block == B200_BLOCK_LAYERNORM) {
             ly::BlockNormArgs a = ly_block_norm_args(Y);
             a.w1 = Y.final_norm; a.b1 = Y.final_norm_b; a.gather = Y.rows;
             a.out1_32 = Y.f32 ? Y.A32 : nullptr; a.out1_16 = Y.f32 ? nullptr : Y.A16;
-            if ((rc = launch_k(p, false, ly::k_block_norm_rows, dim3(m), dim3(LY_NORM_THREADS), (size_t)E * 4, a))) return rc;
+            if ((rc = ly_launch_block_norm(p, m, a))) return rc;
         } else {
             ly::NormArgs a{};
             a.x = Y.X; a.w_pre = Y.final_norm; a.gather = Y.rows; a.eps = Y.c.norm_eps; a.E = E; a.w_off = Y.w_off;
@@ -998,7 +1048,7 @@ static int ly_kv_reset(b200_plan *p) {
     for (LyRun &R : Y.runs) {
         if (R.S) {
             CK(cudaMemsetAsync(R.S, 0, R.s_floats * 4, p->stream));
-            CK(cudaMemsetAsync(R.cstate, 0, R.c_floats * 4, p->stream));
+            if (R.cstate) CK(cudaMemsetAsync(R.cstate, 0, R.c_floats * 4, p->stream));
         }
         if (R.prev) CK(cudaMemsetAsync(R.prev, 0, (size_t)Y.c.width * 4, p->stream));
         if (!R.own || !R.kc) continue;
@@ -1027,6 +1077,7 @@ static int ly_read_buffer(b200_plan *p, const char *name, int layer, void *dst, 
         if (layer < 0 || layer >= (int)Y.runs.size() || !Y.runs[layer].S) return fail(p, B200_ERR_BAD_ARG, "run %d has no %s", layer, name);
         src = s == "delta_state" ? Y.runs[layer].S : Y.runs[layer].cstate;
         sz = (s == "delta_state" ? Y.runs[layer].s_floats : Y.runs[layer].c_floats) * 4;
+        if (!src) return fail(p, B200_ERR_BAD_ARG, "run %d has no %s", layer, name);
     } else return fail(p, B200_ERR_BAD_ARG, "unknown buffer %s", name);
     if (bytes < sz) sz = bytes;
     CK(cudaSetDevice(p->device));
@@ -1047,7 +1098,7 @@ static int ly_time_kernel(b200_plan *p, int which, int reps, float *avg_ms, int6
     auto one = [&](const LyLayer *L) -> int {
         switch (which) {
         case 0: if (!L->w_gu) return B200_OK; bytes = (int64_t)2 * L->s.ff_dim * E * 2; launches++;
-                if (L->s.ff_kind == B200_FF_DENSE_PLAIN) { // one matrix, activation in the epilogue
+                if (L->s.ff_kind == B200_FF_DENSE_PLAIN || L->s.moe_plain) { // one matrix, activation in the epilogue
                     bytes /= 2;
                     return ly_project<ly::EPI_ACT>(p, true, 1, Y.A32, nullptr, L->w_gu, nullptr, L->s.ff_dim, E, Y.H32, nullptr, L->s.ff_dim, L->s.ff_act);
                 }

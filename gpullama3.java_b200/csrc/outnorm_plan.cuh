@@ -426,21 +426,11 @@ static int ly_enqueue_outnorm(b200_plan *p, bool decode, int n, const StepState 
                 nl++;
                 pend.y = Y.Y;
             } else {
-                const int F = s.ff_dim, X = s.ff_experts, XI = X + s.moe_identity, top = s.ff_top, SF = s.moe_shared_ff;
+                const int X = s.ff_experts, XI = X + s.moe_identity, top = s.ff_top, SF = s.moe_shared_ff;
                 const int groups = XI > X ? X + 1 : X; // the identity experts share one id behind the real ones
-                const ly::RouteMode rm{1, L.correction, X, s.moe_scale};
+                const ly::RouteMode rm{1, L.correction, X, s.moe_scale, nullptr};
                 const int extra = SF > 0 ? 1 : 0;
-                if (decode) { // one row: the router's rows stream through the multi-CTA matvec, one warp selects
-                    if ((rc = ly_project<ly::EPI_STORE>(p, true, 1, x32, nullptr, L.w_router, nullptr, XI + extra, E, Y.ZR, nullptr, XI + extra, 0))) return rc;
-                    if ((rc = launch_k(p, false, ly::k_moe_topk, dim3(1), dim3(32), (size_t)2 * XI * 4, (const float *)Y.ZR, XI, top, Y.moe_ids, Y.moe_wts, rm))) return rc;
-                    nl += 2;
-                } else {
-                    const size_t rsm = (size_t)(E + 2 * (XI + extra)) * 4;
-                    if (h16) rc = launch_k(p, false, ly::k_moe_route<ly::bf16>, dim3(n), dim3(128), rsm, (const ly::bf16 *)Y.A16, (const ly::bf16 *)L.w_router, n, E, XI, top, 1, Y.moe_ids, Y.moe_wts, rm, extra, Y.SGL);
-                    else rc = launch_k(p, false, ly::k_moe_route<float>, dim3(n), dim3(128), rsm, x32, (const ly::bf16 *)L.w_router, n, E, XI, top, 1, Y.moe_ids, Y.moe_wts, rm, extra, Y.SGL);
-                    if (rc) return rc;
-                    nl++;
-                }
+                if ((rc = ly_enqueue_route(p, decode, n, L, x32, Y.A16, XI, extra, rm, &nl))) return rc;
                 if (SF > 0) { // the shared expert runs for every row; its hidden rows leave the buffer before the experts use it
                     LyTc t_sgu, t_sdown;
                     if (Y.tc && !decode) {
@@ -454,42 +444,8 @@ static int ly_enqueue_outnorm(b200_plan *p, bool decode, int n, const StepState 
                 }
                 pend.ids = Y.moe_ids; pend.wts = Y.moe_wts; pend.top = top; pend.n_real = X;
                 pend.ys = Y.YS; // never read when every chosen expert is an identity
-                if (X > 0 && h16 && Y.tc && L.tc_moe) {
-                    // tcgen05 route: slots sorted by expert, every expert padded to whole 128-row tiles (identity slots get no row); the
-                    // routing weight multiplies the experts' results in the row kernel
-                    int t128 = (n * top + 127) / 128 + X;
-                    if (t128 > Y.max_tiles128) t128 = Y.max_tiles128;
-                    if ((rc = launch_k(p, false, ly::k_moe_group_padded, dim3(1), dim3(1024), (size_t)3 * groups * 4, (const int *)Y.moe_ids, (const float *)Y.moe_wts, n * top, groups, t128, Y.srt,
-                                       Y.slot_row, Y.row_scale, Y.tile_group128, X, 1))) return rc;
-                    if ((rc = launch_k(p, false, ly::k_moe_gather, dim3(t128 * 128), dim3(128), (size_t)0, (const ly::bf16 *)Y.A16, E, top, (const int *)Y.srt, (const int *)Y.tile_group128, Y.AS16))) return rc;
-                    const uint32_t fl = pg::FLAVOR_BF16 | pg::FLAVOR_SILU_BF16;
-                    int gr = pg::gemm_launch<pg::GEMM_GATEUP, pg::GEMM_STAGES>(Y.m_as, L.m_moe_gate, L.m_moe_up, Y.m_ysp, Y.HS16, F, t128 * 128, t128, F / (pg::BN / 2), E, p->stream, fl,
-                                                                             pg::Grouped{Y.tile_group128, 2 * F, nullptr});
-                    if (!gr) gr = pg::gemm_launch<pg::GEMM_F32, pg::GEMM_STAGES>(L.m_moe_h, L.m_moe_down, L.m_moe_down, Y.m_ysp, Y.YSP, E, t128 * 128, t128, E / pg::BN, F, p->stream, pg::FLAVOR_BF16,
-                                                                                pg::Grouped{Y.tile_group128, E, nullptr});
-                    if (gr) return fail(p, B200_ERR_CUDA, "tensor-core expert GEMM launch failed (%d)", gr);
-                    nl += 4;
-                    pend.ys = Y.YSP; pend.ys_map = Y.slot_row;
-                } else if (X > 0) {
-                    int tiles = 0;
-                    if (!decode) {
-                        tiles = (n * top + 63) / 64 + groups;
-                        if (tiles > Y.max_tiles) tiles = Y.max_tiles;
-                        if ((rc = launch_k(p, false, ly::k_moe_group, dim3(1), dim3(1024), (size_t)3 * groups * 4, (const int *)Y.moe_ids, n * top, groups, tiles, Y.moe_perm, Y.tile_group, Y.tile_row0,
-                                           Y.tile_rows, X))) return rc;
-                        nl++;
-                    }
-                    ly::GemmView gv{};
-                    ly::MvView mv{};
-                    gv.tile_group = Y.tile_group; gv.tile_row0 = Y.tile_row0; gv.tile_rows = Y.tile_rows; gv.perm = Y.moe_perm;
-                    gv.a_div = top; gv.w_gs = mv.w_gs = (long long)2 * F * E;
-                    mv.group = Y.moe_ids; mv.y_bs = F; mv.n_groups = X;
-                    if ((rc = ly_project_view<ly::EPI_GATED>(p, decode, n, x32, Y.A16, L.w_gu, F, E, Y.H32, h16 ? Y.H16 : nullptr, F, s.ff_act, gv, mv, top, 1, tiles))) return rc;
-                    gv.a_div = 1; gv.w_gs = mv.w_gs = (long long)E * F;
-                    mv.x_bs = F; mv.y_bs = E;
-                    if ((rc = ly_project_view<ly::EPI_STORE>(p, decode, n, Y.H32, Y.H16, L.w_down, E, F, Y.YS, nullptr, E, 0, gv, mv, top, 1, tiles))) return rc;
-                    nl += 2;
-                }
+                // the routing weight multiplies the experts' results in the row kernel
+                if (X > 0 && (rc = ly_enqueue_experts(p, decode, n, L, x32, Y.A16, groups, false, &pend.ys, &pend.ys_map, &nl))) return rc;
             }
             pend.w = L.norm2; pend.ls = L.ls2;
         }

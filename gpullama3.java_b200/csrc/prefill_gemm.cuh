@@ -21,7 +21,8 @@ constexpr int BM = 128, BK = 64, BN = 128;
 // Epilogue modes: F32 store (QKV), F32 read-add-store (x += A*W^T: Wo and W2), and the gate/up pair:
 // the B tile is 64 rows of W1 and 64 rows of W3 for the same 64 hidden units, so accumulator columns
 // [0,64) = gate, [64,128) = up, and the epilogue emits f16(silu(gate)*up) (InferenceCore.java:150-158).
-enum { GEMM_F32 = 0, GEMM_RESID = 1, GEMM_GATEUP = 2 };
+// GEMM_ACT (single-CTA kernel): a plain product with an activation, bf16(act(C)).
+enum { GEMM_F32 = 0, GEMM_RESID = 1, GEMM_GATEUP = 2, GEMM_ACT = 3 };
 
 __device__ __forceinline__ uint32_t s32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t cnt) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(cnt)); }
@@ -59,7 +60,8 @@ constexpr uint32_t UMMA_IDESC_AB_BF16 = (1u << 7) | (1u << 10);
 //   FLAVOR_GELU_BF16  the gate/up epilogue emits bf16(gelu_tanh(g) * u) instead of f16(silu(g) * u).
 //   FLAVOR_SILU_BF16  the gate/up epilogue emits bf16(silu(g) * u).
 //   FLAVOR_RELU_BF16  the gate/up epilogue emits bf16(max(g, 0) * u).
-enum { FLAVOR_BF16 = 1u, FLAVOR_GELU_BF16 = 2u, FLAVOR_SILU_BF16 = 4u, FLAVOR_RELU_BF16 = 8u };
+//   FLAVOR_RELU2_BF16 the GEMM_ACT epilogue emits bf16(max(c, 0)^2) (without it bf16(c)).
+enum { FLAVOR_BF16 = 1u, FLAVOR_GELU_BF16 = 2u, FLAVOR_SILU_BF16 = 4u, FLAVOR_RELU_BF16 = 8u, FLAVOR_RELU2_BF16 = 16u };
 // Grouped rows (a mixture of experts; single-CTA kernel): the rows of A are sorted by group and every group is padded to whole
 // 128-row tiles, so an M tile belongs to ONE group: tile_group[m tile] (-1: no work) selects the weight matrix, whose rows start
 // b_rows * group further down the B tensor map(s).  row_scale (nullable) multiplies gate and up before the activation (a weight
@@ -84,6 +86,14 @@ __device__ __forceinline__ uint32_t gated_pair(uint32_t flavor, float g0, float 
         return *reinterpret_cast<const uint32_t *>(&hh);
     }
     const __half2 hh = __floats2half2_rn((g0 / (1.0f + expf(-g0))) * u0, (g1 / (1.0f + expf(-g1))) * u1);
+    return *reinterpret_cast<const uint32_t *>(&hh);
+}
+__device__ __forceinline__ uint32_t act_pair(uint32_t flavor, float c0, float c1) {
+    if (flavor & FLAVOR_RELU2_BF16) {
+        c0 = fmaxf(c0, 0.0f); c1 = fmaxf(c1, 0.0f);
+        c0 *= c0; c1 *= c1;
+    }
+    const __nv_bfloat162 hh = __floats2bfloat162_rn(c0, c1);
     return *reinterpret_cast<const uint32_t *>(&hh);
 }
 __host__ __device__ constexpr uint32_t umma_idesc_f16(int m, int n) { return (1u << 4) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24); }
@@ -204,6 +214,24 @@ __global__ void __launch_bounds__(256) k_gemm_f16_tcgen05(const __grid_constant_
                             const float g0 = __uint_as_float(g[8 * v + 2 * e]) * sc, g1 = __uint_as_float(g[8 * v + 2 * e + 1]) * sc;
                             w[e] = gated_pair(flavor, g0, g1, __uint_as_float(u[8 * v + 2 * e]) * sc, __uint_as_float(u[8 * v + 2 * e + 1]) * sc);
                         }
+                        dst[v] = make_uint4(w[0], w[1], w[2], w[3]);
+                    }
+                }
+            }
+        } else if (MODE == GEMM_ACT) {
+            __nv_bfloat16 *C = reinterpret_cast<__nv_bfloat16 *>(Cv);
+#pragma unroll 1
+            for (int c0 = 0; c0 < BN; c0 += 32) {
+                uint32_t r[32];
+                tmem_ld32(tlane + (uint32_t)c0, r);
+                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                if (row < m_valid) {
+                    uint4 *dst = reinterpret_cast<uint4 *>(C + (size_t)row * ldc + n0 + c0);
+#pragma unroll
+                    for (int v = 0; v < 4; v++) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) w[e] = act_pair(flavor, __uint_as_float(r[8 * v + 2 * e]), __uint_as_float(r[8 * v + 2 * e + 1]));
                         dst[v] = make_uint4(w[0], w[1], w[2], w[3]);
                     }
                 }

@@ -25,6 +25,7 @@ ARCH_PIBIDRA = 3
 ARCH_LATUSUN = 4
 ARCH_LEROSUN = 5
 ARCH_DINUZEN = 6
+ARCH_KEGASUN = 7
 
 GGML_BF16 = 30  # ggml's id for bfloat16; layered plans take their safetensors tensors under it
 _SAFETENSORS_TYPES = {"BF16": GGML_BF16, "F16": GGMLType.F16, "F32": GGMLType.F32}
@@ -102,9 +103,13 @@ class LayerSpec:
     mixer_norm_groups: int = 1
     # mixture of experts
     moe_router: str = "sigmoid_input"   # | "softmax_output": softmax scores, selection by score + correction, weights on the outputs
+    #                                     | "softmax_chosen": selection by logit + bias, softmax over the chosen logits on the outputs
     moe_identity: int = 0               # identity experts behind the real ones
     moe_scale: float = 1.0
     moe_shared_ff: int = 0              # width of the shared expert (0: none)
+    moe_plain: bool = False             # experts without a gate: down(act(up x))
+    q_rank: int = 0                     # latent attention: > 0: queries through a normed latent of that size
+    gate_cap: float = 0.0               # "mlstm": soft cap of both gates' logits
 
 
 @dataclass
@@ -128,6 +133,9 @@ class LayeredConfiguration:
     norm_groups: int = 1
     token_shift: bool = False
     depth_average: bool = False
+    # "layernorm": x += mixer(LN x); x += ff(LN x), layer norms with a weight and no bias
+    bigram: tuple | None = None  # (buckets, factor of the previous token, factor of the token): a hashed row added to the embedding
+    sinusoid_base: float = 0.0   # > 0: a sinusoidal position vector added to the embedding
 
     @property
     def n_layers(self):
@@ -329,9 +337,45 @@ def dinuzen_configuration(cfg: dict, tensor_shapes: dict, context_length: int) -
         block="outnorm", norm_groups=int(cfg["norm"].get("groups", 1)), token_shift=True, depth_average=True)
 
 
+def kegasun_configuration(cfg: dict, tensor_shapes: dict, context_length: int) -> LayeredConfiguration:
+    """config.json of a Kegasun model -> LayeredConfiguration: pre-norm blocks with layer norms over an embedding with bigram rows and
+    sinusoidal positions; per layer a sliding-window latent attention (low-rank queries, learned sink, per-head gate) or a matrix memory
+    (mLSTM), and a gated SiLU feed-forward, a mixture of plain squared-ReLU experts, or none.  All sizes and all model-dependent
+    constants are read from the file."""
+    layers = []
+    for i, lc in enumerate(cfg["layers"]):
+        m, mlp = lc["mixer"], lc.get("mlp")
+        if mlp is None:
+            ff = dict(ff_dim=0)
+        elif mlp.get("kind") == "dense":
+            ff = dict(ff_dim=int(mlp["ff"]), ff_act="silu")
+        elif mlp.get("kind") == "moe":
+            r = mlp["router"]
+            ff = dict(ff_dim=int(mlp["expert"]["ff"]), ff_act="relu2", ff_kind="moe", ff_experts=int(r["experts"]), ff_top=int(r["top"]),
+                      moe_router="softmax_chosen", moe_plain=True)
+        else:
+            raise UnsupportedModel(f"layer {i}: feed-forward kind {mlp.get('kind')!r}")
+        base = dict(heads=int(m["heads"]), key_dim=int(m["dim"]), value_dim=int(m["vdim"]), bias_rows=0, bias_far=0.0, softcap=0.0, qkv_bias=False, qk_norm=False)
+        if lc["type"] == "latent_attention":
+            mask = m.get("mask")
+            layers.append(LayerSpec(kv_heads=1, window=int(mask["size"]) if mask else int(context_length), score_scale=float(m["scale"]), sink=True, sink_learned=True,
+                                    gate=True, gate_per_head=True, mixer="latent_attention", kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]), **base, **ff))
+        elif lc["type"] == "mlstm":
+            layers.append(LayerSpec(kv_heads=int(m["heads"]), window=1, score_scale=float(int(m["dim"]) ** -0.5), sink=False, gate=True, mixer="mlstm",
+                                    gate_cap=float(m["gate_cap"]), **base, **ff))
+        else:
+            raise UnsupportedModel(f"layer {i}: mixer type {lc['type']!r} (Kegasun layers are 'latent_attention' or 'mlstm')")
+    emb = cfg["embedding"]
+    bg = emb.get("bigram")
+    return LayeredConfiguration(
+        ARCH_KEGASUN, int(cfg["width"]), int(cfg["vocab"]), int(context_length), float(cfg["norm"]["eps"]), float(emb.get("scale", 1.0)), layers, None,
+        block="layernorm", bigram=(int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])) if bg else None, sinusoid_base=10000.0)
+
+
 # config.json "architecture" -> (model type, configuration builder): the registry of safetensors model directories
 CONFIG_ARCHITECTURES = {"Pibidra": ("PIBIDRA", pibidra_configuration), "Latusun": ("LATUSUN", latusun_configuration),
-                        "Lerosun": ("LEROSUN", lerosun_configuration), "Dinuzen": ("DINUZEN", dinuzen_configuration)}
+                        "Lerosun": ("LEROSUN", lerosun_configuration), "Dinuzen": ("DINUZEN", dinuzen_configuration),
+                        "Kegasun": ("KEGASUN", kegasun_configuration)}
 DEFAULT_LAYERED_CONTEXT = 4096
 
 

@@ -43,7 +43,7 @@ class LayerSpec(C.Structure):
                [(n, C.c_int32) for n in ("ff_experts", "ff_top", "value_from_key", "head_temp", "head_mix", "conv_taps", "score_maps")] + \
                [("diff_init", C.c_float)] + \
                [(n, C.c_int32) for n in ("qk_head_norm", "mixer_norm_groups", "moe_router", "moe_identity")] + \
-               [("moe_scale", C.c_float), ("moe_shared_ff", C.c_int32)]
+               [("moe_scale", C.c_float), ("moe_shared_ff", C.c_int32), ("q_rank", C.c_int32), ("gate_cap", C.c_float), ("moe_plain", C.c_int32)]
 
 
 class LayeredConfig(C.Structure):
@@ -51,16 +51,17 @@ class LayeredConfig(C.Structure):
                [("norm_eps", C.c_float), ("embedding_scale", C.c_float)] + \
                [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "compute", "block")] + \
                [("residual_mult", C.c_float), ("logit_softcap", C.c_float)] + \
-               [(n, C.c_int32) for n in ("norm_groups", "token_shift", "depth_average")]
+               [(n, C.c_int32) for n in ("norm_groups", "token_shift", "depth_average", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "sinusoid")] + \
+               [("sinusoid_base", C.c_float)]
 
 
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
-ACTIVATIONS = {"gelu_tanh": 0, "silu": 1, "relu": 2, "gelu_erf": 3}
-MIXERS = {"window_attention": 1, "latent_attention": 2, "gated_delta": 3, "rglru": 4, "ssd": 5}
+ACTIVATIONS = {"gelu_tanh": 0, "silu": 1, "relu": 2, "gelu_erf": 3, "relu2": 4}
+MIXERS = {"window_attention": 1, "latent_attention": 2, "gated_delta": 3, "rglru": 4, "ssd": 5, "mlstm": 6}
 FF_KINDS = {"none": 0, "dense": 1, "moe": 2, "dense_plain": 3}
-MOE_ROUTERS = {"sigmoid_input": 0, "softmax_output": 1}
+MOE_ROUTERS = {"sigmoid_input": 0, "softmax_output": 1, "softmax_chosen": 2}
 ROPE_LAYOUTS = {"half": 0, "interleaved": 1}
-BLOCKS = {"sandwich": 0, "parallel": 1, "prenorm": 2, "outnorm": 3}
+BLOCKS = {"sandwich": 0, "parallel": 1, "prenorm": 2, "outnorm": 3, "layernorm": 4}
 
 
 class Tensor(C.Structure):

@@ -67,6 +67,10 @@ def make_layered_config(model: Model, compute: str = "bfloat16"):
     cfg.compute = {"bfloat16": native.COMPUTE_BF16, "bf16": native.COMPUTE_BF16, "float32": native.COMPUTE_F32, "f32": native.COMPUTE_F32}[compute]
     cfg.block, cfg.residual_mult, cfg.logit_softcap = native.BLOCKS[c.block], c.residual_mult, c.logit_softcap
     cfg.norm_groups, cfg.token_shift, cfg.depth_average = c.norm_groups, int(c.token_shift), int(c.depth_average)
+    if c.bigram is not None:  # factors modulo the bucket count: the same row, and always in the range of 32-bit integers
+        b, mp, mc = c.bigram
+        cfg.bigram_buckets, cfg.bigram_mul_prev, cfg.bigram_mul_cur = b, mp % b, mc % b
+    cfg.sinusoid, cfg.sinusoid_base = int(c.sinusoid_base > 0.0), c.sinusoid_base
     specs = []
     for s in c.layers:
         if s.mixer not in native.MIXERS:
@@ -87,6 +91,7 @@ def make_layered_config(model: Model, compute: str = "bfloat16"):
         sp.yarn_factor, sp.yarn_original, sp.yarn_fast, sp.yarn_slow = s.yarn
         sp.score_maps, sp.diff_init, sp.qk_head_norm, sp.mixer_norm_groups = s.score_maps, s.diff_init, int(s.qk_head_norm), s.mixer_norm_groups
         sp.moe_router, sp.moe_identity, sp.moe_scale, sp.moe_shared_ff = native.MOE_ROUTERS[s.moe_router], s.moe_identity, s.moe_scale, s.moe_shared_ff
+        sp.q_rank, sp.gate_cap, sp.moe_plain = s.q_rank, s.gate_cap, int(s.moe_plain)
         specs.append(sp)
     return cfg, specs
 

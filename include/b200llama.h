@@ -63,6 +63,11 @@ extern "C" {
                              * subtracted), which may read another layer's keys and values; the feed-forward is a plain GELU layer or a
                              * softmax-routed mixture of gated SiLU experts with identity experts and a gated shared expert */
 
+#define B200_ARCH_KEGASUN 7 /* a layered design: pre-norm blocks x += mixer(LN x); x += ff(LN x) with layer norms (weight, no bias) over an embedding that adds
+                             * a hashed bigram row and a sinusoidal position vector; mixers: sliding-window latent attention with low-rank queries, a
+                             * learned sink and a gate per head, or a matrix memory with exponential gates (mLSTM); feed-forward: gated SiLU or a
+                             * mixture of plain squared-ReLU experts weighted by the softmax over the chosen logits */
+
 /* GGML tensor type ids accepted for weights (tensor/GGMLType.java:5-20) */
 #define B200_GGML_F32 0
 #define B200_GGML_F16 1
@@ -145,6 +150,11 @@ int b200_plan_create(const b200_config *cfg, const b200_tensor *tensors, int32_t
                             * h / (heads / kv_heads)) a state S [key_dim][value_dim]: S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x;
                             * y * silu(z) is RMS-normed in mixer_norm_groups parts times ".norm", then W_o.  S (FP32) and the last conv_taps - 1
                             * convolution inputs are carried between calls */
+#define B200_MIXER_MLSTM 6 /* q = W_q a * key_dim^-1/2, k = W_k a (heads x key_dim), v = W_v a (heads x value_dim); per head log input gate i = C
+                            * tanh((W_i a + ".i.b") / C), log forget gate f = log sigmoid(C tanh((W_f a + ".f.b") / C)), C = gate_cap; state S [key_dim]
+                            * [value_dim], n [key_dim], m, all zero at position 0: m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, n
+                            * likewise with k alone; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6); o / rms(o) per head, times ".norm" [heads * value_dim]
+                            * times sigmoid(W_g a), then W_o.  The state is FP32 and carried between calls */
 #define B200_FF_NONE 0
 #define B200_FF_DENSE_GATED 1 /* down(act(gate x) * (up x)) */
 #define B200_FF_MOE 2         /* sum over the ff_top experts with the largest router scores of expert_e(s_e * x), expert = FF_DENSE_GATED without
@@ -154,6 +164,7 @@ int b200_plan_create(const b200_config *cfg, const b200_tensor *tensors, int32_t
 #define B200_MOE_SOFTMAX_OUTPUT 1 /* s = softmax(z) over experts + identity experts; the `top` largest of s + "<layer>.mlp.correction" are chosen;
                                    * weights s / (sum of the chosen s + 1e-20) * moe_scale multiply the experts' OUTPUTS; the last moe_identity router
                                    * outputs belong to identity experts, which return what they read and own no tensors */
+#define B200_MOE_SOFTMAX_CHOSEN 2 /* z + "<layer>.mlp.router.b"; the `top` largest; weights = softmax over the chosen logits, on the experts' OUTPUTS */
 #define B200_ROPE_HALF 0        /* pair (i, i + rot_dims / 2) */
 #define B200_ROPE_INTERLEAVED 1 /* pair (2i, 2i + 1) */
 #define B200_BLOCK_SANDWICH 0 /* x += N(mixer(N x)); x += N(ff(N x)) with (1 + w)-weighted RMS norms (Pibidra) */
@@ -166,10 +177,12 @@ int b200_plan_create(const b200_config *cfg, const b200_tensor *tensors, int32_t
                                * sequence's state in every layer); depth_average: behind layer i, x <- sum_{j <= i+1} "<layer>.dwa"[j] X_j with X_0
                                * what the embedding gave and X_(i+1) what layer i left before it was averaged.  The final norm is the grouped one too */
 #define B200_BLOCK_PARALLEL 1 /* x += residual_mult * (mixer(LN1 x) + ff(LN2 x)), layer norms with weight and bias ("<layer>.norm1", ".norm1.b", ...) */
+#define B200_BLOCK_LAYERNORM 4 /* x += mixer(LN(x; w1)); x += ff(LN(x; w2)), layer norms with a weight and no bias ("<layer>.norm1", ".norm2"; "final.norm") */
 #define B200_ACT_GELU_TANH 0
 #define B200_ACT_SILU 1
 #define B200_ACT_RELU 2
 #define B200_ACT_GELU_ERF 3
+#define B200_ACT_RELU2 4 /* max(z, 0)^2 */
 #define B200_COMPUTE_BF16 0 /* prefill GEMM operands rounded to BF16, FP32 accumulation; decode FP32 activations x BF16 weights */
 #define B200_COMPUTE_F32 1  /* every product in true FP32 (BF16 weights widen exactly) */
 
@@ -229,10 +242,17 @@ typedef struct b200_layer_spec {
     float moe_scale;
     int32_t moe_shared_ff;  /* > 0: a shared expert of that width ("<layer>.mlp.shared.{gate,up,down}") is evaluated for all tokens and added times
                                sigmoid(<"<layer>.mlp.shared.sg", x>) */
+    /* B200_MIXER_LATENT_ATTENTION in a B200_BLOCK_LAYERNORM plan (window, sink and gate as for windowed attention; rot_dim = 0) */
+    int32_t q_rank;         /* > 0: queries through a latent of their own, q = Wuq (RMS norm(Wdq a) * "<layer>.mix.dq.norm") ("<layer>.mix.dq" [q_rank][width],
+                               ".uq" [heads * key_dim][q_rank]); 0: q = Wq a */
+    /* B200_MIXER_MLSTM */
+    float gate_cap;
+    /* B200_FF_MOE */
+    int32_t moe_plain;      /* 1: experts without a gate, down(act(up x)) ("<layer>.mlp.e<k>.{up,down}") */
 } b200_layer_spec;
 
 typedef struct b200_layered_config {
-    int32_t arch;           /* B200_ARCH_PIBIDRA, B200_ARCH_LATUSUN, B200_ARCH_LEROSUN, B200_ARCH_DINUZEN */
+    int32_t arch;           /* B200_ARCH_PIBIDRA, B200_ARCH_LATUSUN, B200_ARCH_LEROSUN, B200_ARCH_DINUZEN, B200_ARCH_KEGASUN */
     int32_t width;
     int32_t vocab_size;
     int32_t n_layers;
@@ -247,6 +267,12 @@ typedef struct b200_layered_config {
     int32_t norm_groups;    /* B200_BLOCK_OUTNORM: parts of every residual norm (>= 1; 0 reads as 1) */
     int32_t token_shift;    /* B200_BLOCK_OUTNORM: 1 = the mixers read the shifted row */
     int32_t depth_average;  /* B200_BLOCK_OUTNORM: 1 = the depth average behind every layer */
+    int32_t bigram_buckets; /* B200_BLOCK_LAYERNORM, > 0: the embedding adds row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod
+                               bigram_buckets of "bigram" [bigram_buckets + 1][width]; a sequence's first token takes the last row.  The tokens of earlier
+                               calls are part of the sequence's state */
+    int32_t bigram_mul_prev, bigram_mul_cur;
+    int32_t sinusoid;       /* B200_BLOCK_LAYERNORM, 1: the embedding adds sin(p base^(-2i / width)) to entry 2i and its cos to entry 2i + 1 */
+    float sinusoid_base;
 } b200_layered_config;
 
 /* prefill_batch_size = the most tokens one b200_forward_batch_prefill / _batch_logits call takes (>= 1). */
