@@ -392,6 +392,78 @@ def compare_dinuzen(pkg, lb, local: int, steps: int, warmup: int, sizes):
             "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "tensor_tflops": burst, "tensor_source": t_src}, "sizes": out}
 
 
+# ---- --compare kegasun: the layer-norm hybrid (windowed latent attention with query latents, matrix memory, plain experts) beside the two
+# existing models it is closest to at equal size: Latusun (latent attention over the same latent, every layer a mixture of experts) and
+# Dinuzen (a recurrence with a matrix state of as many entries, attention, the same kinds of feed-forward).  Same width, vocabulary, number
+# of layers, heads, key / value / latent sizes, state entries and weights per expert and dense feed-forward (plain experts carry two
+# matrices, gated ones three: their widths are in the ratio 3 : 2).
+KEGASUN_SIZES = {
+    # width, attention heads, key = value size, query latent, key/value latent, window, memory heads, memory key, memory value, experts, chosen, expert ff, dense ff, vocab
+    "small": (1024, 16, 64, 384, 256, 512, 4, 128, 256, 8, 2, 1536, 2816, 32768),
+    "1b-like": (2048, 16, 128, 768, 512, 512, 8, 128, 256, 16, 4, 2304, 5632, 32768),
+}
+
+
+def kegasun_compare_models(S, name: str):
+    """(Kegasun config, Latusun config, Dinuzen config, accounting) of one compare size."""
+    E, H, d, Rq, R, W, MH, mk, mv, X, top, F, DF, V = KEGASUN_SIZES[name]
+    moe, dense = S.kegasun_moe(X, top, F), S.kegasun_dense(DF)
+    cfg = S.kegasun_config(E, V, [S.kegasun_mlstm(MH, mk, mv, moe), S.kegasun_attention(H, d, d, Rq, R, W, dense), S.kegasun_mlstm(MH, mk, mv, dense),
+                                  S.kegasun_attention(H, d, d, Rq, R, W, moe)], bigram=(65521, 31, 17))
+    FG = F * 2 // 3
+    A, B = "latent_attention", "latent_attention_2"
+    lcfg = S.latusun_config(E, V, [S.latusun_layer(k, H, d - d // 4, d // 4, d, R, experts=X, top=top, ff=FG) for k in (A, B, B, A)])
+    dmoe, ddense = S.dinuzen_moe(X, top, FG), S.dinuzen_dense(DF * 3 // 2)
+    SP, SN = 64, mk  # state entries: SH * SP * SN = MH * mk * mv
+    SH = MH * mv // SP
+    dcfg = S.dinuzen_config(E, V, [S.dinuzen_mamba2(SH, SP, SN, 1, 4, dmoe), S.dinuzen_attention(H // 2, 2, d, d, ddense), S.dinuzen_mamba2(SH, SP, SN, 1, 4, ddense),
+                                   S.dinuzen_attention(H // 2, 2, d, d, dmoe)])
+    w_moe, w_dense = X * E + top * 2 * F * E, 3 * DF * E
+    w_att = (Rq + R + H) * E + H * d * (Rq + 2 * R) + H * d * E
+    w_mem = (2 * MH * mk + 2 * MH * mv + 2 * MH) * E + MH * mv * E
+    l_moe = X * E + top * 3 * FG * E
+    l_att = H * d * E + (R + d // 4) * E + H * (d - d // 4) * R + H * d * R + H * d * E
+    d_ssd = (2 * SH * SP + 2 * SN + SH) * E + SH * SP * E
+    d_att = (H + 4) * d * E + 2 * d * E + H // 2 * d * E
+    acct = {"streamed": w_moe * 2 + w_dense * 2 + w_att * 2 + w_mem * 2, "att_mac_per_pair": 2 * H * d, "mem_mac_per_token": 3 * MH * mk * (mv + 1),
+            "l_streamed": 4 * (l_moe + l_att) + 2 * H * d * E, "l_att_mac_per_pair": 2 * H * d,
+            "d_streamed": 2 * (l_moe + w_dense + d_ssd + d_att), "d_att_mac_per_pair": H * 2 * d, "d_ssd_mac_per_token": 3 * SH * SP * SN}
+    return cfg, lcfg, dcfg, acct
+
+
+def compare_kegasun(pkg, lb, local: int, steps: int, warmup: int, sizes):
+    hbm, hbm_src = peaks()
+    burst, sustained, t_src = tensor_peak()
+    S = pkg.synth
+    out = {}
+    for name in sizes:
+        E, V = KEGASUN_SIZES[name][0], KEGASUN_SIZES[name][-1]
+        depth, n_pp = 64, 512
+        ctx = max(depth + steps + warmup + 8, n_pp + 8)
+        toks = np.asarray(lb.synthetic_tokens(V, ctx), dtype=np.int32)
+        cfg, lcfg, dcfg, a = kegasun_compare_models(S, name)
+        pairs = n_pp * (n_pp + 1) // 2
+        row = {}
+        for key, c, weights, model, streamed, flops in (
+                ("kegasun_bfloat16", cfg, S.kegasun_weights, S.kegasun_model, a["streamed"], 2 * a["att_mac_per_pair"] * pairs + 2 * a["mem_mac_per_token"] * n_pp),
+                ("latusun_bfloat16", lcfg, S.latusun_weights, S.latusun_model, a["l_streamed"], 4 * a["l_att_mac_per_pair"] * pairs),
+                ("dinuzen_bfloat16", dcfg, S.dinuzen_weights, S.dinuzen_model, a["d_streamed"], 2 * a["d_att_mac_per_pair"] * pairs + 2 * a["d_ssd_mac_per_token"] * n_pp)):
+            w = weights(c, 1234)
+            plan = pkg.B200MasterPlan.initialize_plan(model(c, w, ctx), prefill_batch_size=n_pp, device=local, compute="bfloat16")
+            row[key] = _layered_leg(plan, toks, depth, warmup, steps, n_pp, hbm, burst, 2 * (streamed + V * E), 2.0 * streamed * n_pp + 2.0 * flops,
+                                    ((0, "up_or_gate_up"), (1, "down"), (2, "fused_projection"), (3, "mixer_out"), (4, "classifier")))
+            plan.free()
+            del w
+        row["config"] = {"width": E, "vocab": V, "layers": 4, "order": "matrix memory + experts, attention + dense, matrix memory + dense, attention + experts",
+                         "sizes": dict(zip(("width", "attention_heads", "key_value_size", "query_latent", "latent", "window", "memory_heads", "memory_key", "memory_value", "experts", "chosen",
+                                            "expert_ff", "dense_ff", "vocab"), KEGASUN_SIZES[name])),
+                         "closest": "Latusun: four latent-attention layers with experts over the same latent and heads; Dinuzen: state space, attention, state space, attention with as many state entries",
+                         "decode": f"tg{steps} from depth {depth + warmup}", "prefill": f"pp{n_pp} in one chunk from depth 0"}
+        out[name] = row
+    return {"metric": "kegasun_vs_closest_models", "unit": "tok/s", "data": "synthetic", "dtype": "bf16 weights, f32 accumulate",
+            "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "tensor_tflops": burst, "tensor_source": t_src}, "sizes": out}
+
+
 class ClockSampler:
     """nvidia-smi clocks/throttle reasons sampled DURING the timed region."""
     Q = "clocks.sm,clocks.max.sm,power.draw,clocks_event_reasons.hw_slowdown,clocks_event_reasons.hw_thermal_slowdown," \
@@ -507,10 +579,10 @@ def main():
     ap.add_argument("--depth", type=int, default=-1, help="LlamaBench -d: KV positions filled before the timed steps (default: the warm-up steps)")
     ap.add_argument("--workload", default=WORKLOAD, choices=["llama-3-8b", "llama-3-70b", "llama-3.2-1b", "qwen3-4b"],
                     help="shape of the synthetic model (default: the BASELINE headline, Llama-3-8B; 70B is BASELINE config 5, meant for --gpus 2/4/8)")
-    ap.add_argument("--compare", default=None, choices=["pibidra", "latusun", "lerosun", "dinuzen"],
+    ap.add_argument("--compare", default=None, choices=["pibidra", "latusun", "lerosun", "dinuzen", "kegasun"],
                     help="instead of the headline workload: decode and prefill throughput of a layered design beside its closest existing model "
-                         "at equal sizes (pibidra: the FP16 Qwen3 plan; latusun, lerosun: the Pibidra plan; dinuzen: the Lerosun plan), with per-kernel rooflines; one JSON line")
-    ap.add_argument("--compare-sizes", default=None, help="comma-separated size names (pibidra: 1b-like,8b-like; latusun: small,lite-like; lerosun, dinuzen: small,1b-like)")
+                         "at equal sizes (pibidra: the FP16 Qwen3 plan; latusun, lerosun: the Pibidra plan; dinuzen: the Lerosun plan; kegasun: the Latusun and the Dinuzen plan), with per-kernel rooflines; one JSON line")
+    ap.add_argument("--compare-sizes", default=None, help="comma-separated size names (pibidra: 1b-like,8b-like; latusun: small,lite-like; lerosun, dinuzen, kegasun: small,1b-like)")
     args = ap.parse_args()
     K, W = args.steps, max(args.warmup, 3)
     if args.compare:
@@ -521,7 +593,9 @@ def main():
         pkg = ge.import_package()
         sampler = ClockSampler(local)
         sampler.start()
-        if args.compare == "dinuzen":
+        if args.compare == "kegasun":
+            line = compare_kegasun(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))
+        elif args.compare == "dinuzen":
             line = compare_dinuzen(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))
         elif args.compare == "lerosun":
             line = compare_lerosun(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))

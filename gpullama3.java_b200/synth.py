@@ -739,3 +739,92 @@ def dinuzen_model(cfg: dict, weights: dict, context_length: int):
     tensors = {k: (loader.GGML_BF16, tuple(reversed(v.shape)), bf16_bits(v).view(np.uint8).reshape(-1)) for k, v in weights.items()}
     config = loader.dinuzen_configuration(cfg, {k: v.shape for k, v in weights.items()}, context_length)
     return loader.Model(None, config, "DINUZEN", tensors)
+
+
+# ---- Kegasun: layer-norm blocks of latent attention and matrix memory over bigram + sinusoidal embeddings --------------------------
+def kegasun_attention(heads: int, key_dim: int, value_dim: int, q_rank: int, kv_rank: int, window: int, mlp: dict | None = None, scale: float | None = None) -> dict:
+    """A sliding-window latent-attention entry of config.json's "layers" (mlp = None: no feed-forward)."""
+    return {"type": "latent_attention",
+            "mixer": {"heads": heads, "dim": key_dim, "vdim": value_dim, "q_rank": q_rank, "kv_rank": kv_rank, "mask": {"size": window},
+                      "scale": float(key_dim ** -0.5 if scale is None else scale)},
+            "mlp": mlp}
+
+
+def kegasun_mlstm(heads: int, key_dim: int, value_dim: int, mlp: dict | None = None, gate_cap: float = 15.0) -> dict:
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": key_dim, "vdim": value_dim, "gate_cap": float(gate_cap)}, "mlp": mlp}
+
+
+def kegasun_dense(ff: int) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def kegasun_moe(experts: int, top: int, ff: int) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def kegasun_config(width: int, vocab: int, layers: list, eps: float = 1e-5, scale: float = 0.75, bigram: tuple | None = (101, 7, 5)) -> dict:
+    """bigram = (buckets, factor of the previous token, factor of the token) or None."""
+    emb = {"scale": float(scale)}
+    if bigram is not None:
+        emb["bigram"] = {"buckets": bigram[0], "mul_prev": bigram[1], "mul_cur": bigram[2]}
+    return {"architecture": "Kegasun", "width": width, "vocab": vocab, "embedding": emb, "norm": {"eps": float(eps)}, "layers": layers}
+
+
+def kegasun_weights(cfg: dict, seed: int = 0) -> dict:
+    """name -> float32 array in the shapes the loader expects (linear weights [out][in]); BF16-representable values."""
+    from .safetensors import bf16_bits, bf16_to_f32
+
+    rng = np.random.default_rng(seed)
+    E, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def mat(o, i, gain=1.0):
+        return (rng.standard_normal((o, i)) * gain / np.sqrt(i)).astype(np.float32)
+
+    def vec(n, mean=0.0, std=1.0):
+        return (mean + std * rng.standard_normal(n)).astype(np.float32)
+
+    w["embed"] = rng.standard_normal((V, E)).astype(np.float32)
+    if cfg["embedding"].get("bigram"):
+        w["bigram"] = (0.7 * rng.standard_normal((cfg["embedding"]["bigram"]["buckets"] + 1, E))).astype(np.float32)
+    w["final.norm"] = vec(E, 1.0, 0.2)
+    w["head"] = mat(V, E)
+    for i, lc in enumerate(cfg["layers"]):
+        m, p = lc["mixer"], f"l{i}."
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        w[p + "norm1"] = vec(E, 1.0, 0.2)
+        if lc["type"] == "latent_attention":
+            Rq, R = m["q_rank"], m["kv_rank"]
+            w[p + "mix.dq"], w[p + "mix.dq.norm"], w[p + "mix.uq"] = mat(Rq, E), vec(Rq, 1.0, 0.3), mat(H * dk, Rq, 1.5)
+            w[p + "mix.dkv"], w[p + "mix.dkv.norm"] = mat(R, E), vec(R, 1.0, 0.3)
+            w[p + "mix.uk"], w[p + "mix.uv"] = mat(H * dk, R, 1.5), mat(H * dv, R)
+            w[p + "mix.sink"], w[p + "mix.g"] = vec(H, 1.0, 1.0), mat(H, E, 2.0)
+        else:
+            w[p + "mix.q"], w[p + "mix.k"], w[p + "mix.v"] = mat(H * dk, E, 1.5), mat(H * dk, E), mat(H * dv, E)
+            w[p + "mix.i"], w[p + "mix.i.b"] = mat(H, E, 1.5), vec(H, 0.0, 1.0)
+            w[p + "mix.f"], w[p + "mix.f.b"] = mat(H, E, 1.5), vec(H, 3.0, 1.0)
+            w[p + "mix.g"], w[p + "mix.norm"] = mat(H * dv, E, 2.0), vec(H * dv, 1.0, 0.2)
+        w[p + "mix.o"] = mat(E, H * dv)
+        mlp = lc.get("mlp")
+        if mlp is None:
+            continue
+        w[p + "norm2"] = vec(E, 1.0, 0.2)
+        if mlp["kind"] == "dense":
+            F = mlp["ff"]
+            w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = mat(F, E, 1.5), mat(F, E), mat(E, F)
+            continue
+        X, F = mlp["router"]["experts"], mlp["expert"]["ff"]
+        w[p + "mlp.router"], w[p + "mlp.router.b"] = mat(X, E, 1.5), vec(X, 0.0, 0.3)
+        for e in range(X):
+            w[p + f"mlp.e{e}.up"], w[p + f"mlp.e{e}.down"] = mat(F, E), mat(E, F)
+    return {k: bf16_to_f32(bf16_bits(v)).reshape(v.shape) for k, v in w.items()}
+
+
+def kegasun_model(cfg: dict, weights: dict, context_length: int):
+    """In-memory loader.Model (benchmarks and tests: synthetic weights never touch the disk)."""
+    from . import loader
+    from .safetensors import bf16_bits
+
+    tensors = {k: (loader.GGML_BF16, tuple(reversed(v.shape)), bf16_bits(v).view(np.uint8).reshape(-1)) for k, v in weights.items()}
+    config = loader.kegasun_configuration(cfg, {k: v.shape for k, v in weights.items()}, context_length)
+    return loader.Model(None, config, "KEGASUN", tensors)
