@@ -136,7 +136,7 @@ static int ly_enqueue_mlstm(b200_plan *p, bool decode, int n, const StepState *s
     if (rc) return rc;
     const ly::HeadNormArgs ha{L.onorm, s.value_dim, 1, Y.DO + L.gd, s.heads, s.value_dim, Y.c.norm_eps};
     *nl += 2;
-    // one row: a warp's worth of heads per CTA would leave the rest of the device idle either way; a chunk has CTAs enough
+    // one row: eight heads per CTA, a warp each; a chunk has CTAs enough with one per row
     return launch_k(p, false, ly::k_head_norm_gate, dim3(n, decode ? (s.heads + 7) / 8 : 1), dim3(256), (size_t)0, (const float *)Y.DO, Y.maxDO, (const float *)(Y.PROJ + L.g_off), Y.maxP, ha,
                     h16 ? (float *)nullptr : Y.ATT32, h16 ? Y.ATT16 : (ly::bf16 *)nullptr, L.gd);
 }

@@ -368,7 +368,7 @@ int b200_decode_sequence(b200_plan *plan, const int32_t *tokens, int32_t n, int3
 int b200_kv_reset(b200_plan *plan);
 
 /* Test/diagnostic read-back of a named device buffer into host memory.  Names:
- * "x","xb","q","k","v","hb","logits","key_cache","value_cache","xq","xs"; layered plans with a gated-delta run: "delta_state"
+ * "x","xb","q","k","v","hb","logits","key_cache","value_cache","xq","xs"; layered plans with a recurrent run: "delta_state"
  * (the recurrent state of the run, in the recurrence kernel's own order) and "conv_state" (the ring of convolution inputs).  `layer` selects the
  * layer for the KV caches (ignored otherwise).  Copies min(bytes, buffer size).  Layered plans: `layer` is the layer RUN;
  * a latent-attention run has ONE cache, "key_cache" = rows [latent | rotated shared key part], and no "value_cache". */
