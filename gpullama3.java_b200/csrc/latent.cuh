@@ -169,11 +169,6 @@ struct LatentArgs {
     bf16 *cq16;
 };
 
-__device__ __forceinline__ void rope_pair_index(int i, int dims, int layout, int &u, int &v) {
-    if (layout) { u = 2 * i; v = 2 * i + 1; }
-    else { u = i; v = i + dims / 2; }
-}
-
 // cache [ring][rank + dr];  Q [n][heads * (rank + dr)]: this kernel fills the rotated tail of every head, the folded-key
 // product fills the first rank entries;  qu16 (nullable) [n][heads * dk]: BF16 copy of the unrotated query parts.
 // The rotated query parts are also written back into the projection row (the expanded-key prefill reads [q_u | rot q_r] there).
@@ -252,15 +247,18 @@ __global__ void __launch_bounds__(256) k_latent_prep(float *__restrict__ P, int 
 // softmax == 1: scores s = softmax(z) over all router outputs, the `top` largest of s + correction are chosen, weight =
 // s / (sum of the chosen s + 1e-20) * scale.  Router outputs n_real .. are identity experts: they all get the id n_real.
 // softmax == 2: the `top` largest of z + bias, weights = softmax over those chosen values.
+// softmax == 3: weights s = softmax(z) over all experts, not renormalised; the experts form `groups` equal groups of neighbours, a group scores its
+// largest entry, only the `keep` best groups compete (the lowest index wins a tie).
 struct RouteMode {
     int softmax;
     const float *correction; // [experts] (softmax mode)
     int n_real;              // experts with weights (<= experts)
     float scale;
     const float *bias;       // [experts] (mode 2)
+    int groups, keep;        // (mode 3)
 };
 
-// One warp: z [experts] logits in shared memory (overwritten), sbuf [experts] scratch; ids / wts [top] in order of falling choice
+// One warp: z [experts] logits in shared memory (overwritten), sbuf [2 * experts] scratch; ids / wts [top] in order of falling choice
 // score (the lowest index wins a tie).
 __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts, int top, const RouteMode &m, int *ids, float *wts, int lane) {
     if (m.softmax == 2) {
@@ -276,6 +274,33 @@ __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts,
         for (int e = lane; e < experts; e += 32) { const float w = expf(z[e] - mx); sbuf[e] = w; sum += w; }
         sum = warp_sum(sum);
         for (int e = lane; e < experts; e += 32) { const float sc = sbuf[e] / sum; sbuf[e] = sc; z[e] = sc + m.correction[e]; }
+        __syncwarp();
+    }
+    if (m.softmax == 3) { // scores from all logits; the selection runs over the logits themselves (the same order), dropped groups set to -inf
+        float mx = -INFINITY;
+        for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        float sum = 0.0f;
+        for (int e = lane; e < experts; e += 32) { const float w = expf(z[e] - mx); sbuf[e] = w; sum += w; }
+        sum = warp_sum(sum);
+        for (int e = lane; e < experts; e += 32) sbuf[e] /= sum;
+        if (m.keep < m.groups) {
+            float *best = sbuf + experts; // [groups]
+            const int per = experts / m.groups;
+            for (int g = lane; g < m.groups; g += 32) {
+                float b = -INFINITY;
+                for (int i = 0; i < per; i++) b = fmaxf(b, z[g * per + i]);
+                best[g] = b;
+            }
+            __syncwarp();
+            for (int g = lane; g < m.groups; g += 32) {
+                int ahead = 0;
+                for (int k = 0; k < m.groups; k++) ahead += best[k] > best[g] || (best[k] == best[g] && k < g);
+                if (ahead >= m.keep)
+                    for (int i = 0; i < per; i++) z[g * per + i] = -INFINITY;
+            }
+        }
         __syncwarp();
     }
     float tot = 0.0f, z_top = 0.0f;
@@ -312,7 +337,7 @@ __device__ __forceinline__ void route_select(float *z, float *sbuf, int experts,
 // from the same input).  Four warps per CTA: with rows_per_cta == 4 every warp owns a row, with rows_per_cta == 1 the four
 // warps share the rows of one token (what the plan launches: four times the warps in flight, and the kernel is bound by the
 // latency of its loads; the router matrix is small and stays in L2).
-// Dynamic shared memory: rows_per_cta * (E + 2 * (experts + extra)) floats.
+// Dynamic shared memory: rows_per_cta * (E + 3 * (experts + extra)) floats.
 template <typename IN_T>
 __global__ void __launch_bounds__(128) k_moe_route(const IN_T *__restrict__ X, const bf16 *__restrict__ Wr, int n, int E, int experts, int top, int rows_per_cta,
                                                    int *__restrict__ ids, float *__restrict__ wts, RouteMode m, int extra, float *__restrict__ extra_out) {
@@ -320,7 +345,7 @@ __global__ void __launch_bounds__(128) k_moe_route(const IN_T *__restrict__ X, c
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const bool shared_row = rows_per_cta == 1;
     const int r = shared_row ? blockIdx.x : blockIdx.x * 4 + warp;
-    const int zw = 2 * (experts + extra);
+    const int zw = 3 * (experts + extra);
     float *xs = sm + (shared_row ? 0 : (size_t)warp * E), *z = sm + (size_t)rows_per_cta * E + (shared_row ? 0 : (size_t)warp * zw);
     if (r < n) {
         if (shared_row) for (int i = tid; i < E; i += 128) xs[i] = (float)X[(size_t)r * E + i];
@@ -341,7 +366,7 @@ __global__ void __launch_bounds__(128) k_moe_route(const IN_T *__restrict__ X, c
 }
 
 // The decode step spreads the router's rows over several CTAs (k_matvec_bf16) and selects here: one warp, logits z [experts]
-// in, route_select out.  Dynamic shared memory: 2 * experts floats.
+// in, route_select out.  Dynamic shared memory: 3 * experts floats.
 __global__ void __launch_bounds__(32) k_moe_topk(const float *__restrict__ Z, int experts, int top, int *__restrict__ ids, float *__restrict__ wts, RouteMode m) {
     extern __shared__ __align__(16) float z[];
     const int lane = threadIdx.x;

@@ -20,17 +20,17 @@
 #pragma once
 
 // (cos, sin) of every position and rotated pair, evaluated in double: f_i = base^(-2i / dims); with frequency blending
-// f_i <- f_i / factor * ramp_i + f_i * (1 - ramp_i), ramp from pair floor(d(fast)) to ceil(d(slow)) where
+// (linear scaling: all f_i / rope_factor) f_i <- f_i / factor * ramp_i + f_i * (1 - ramp_i), ramp from pair floor(d(fast)) to ceil(d(slow)) where
 // d(t) = dims * ln(original / (2 pi t)) / (2 ln base), and both cos and sin times 0.1 ln(factor) + 1.
 static int ly_rope_table(b200_plan *p, const b200_layer_spec &s, int positions, const float **out) {
     Layered &Y = *p->ly;
-    const std::vector<float> key = {(float)s.rope_dims, s.rope_base, s.yarn_factor, s.yarn_original, s.yarn_fast, s.yarn_slow};
+    const std::vector<float> key = {(float)s.rope_dims, s.rope_base, s.yarn_factor, s.yarn_original, s.yarn_fast, s.yarn_slow, s.rope_factor};
     for (auto &t : Y.rope_tables)
         if (t.first == key) { *out = t.second; return B200_OK; }
     const int dims = s.rope_dims, half = dims / 2;
     std::vector<double> f((size_t)half);
     double mag = 1.0;
-    for (int i = 0; i < half; i++) f[i] = pow((double)s.rope_base, -2.0 * i / dims);
+    for (int i = 0; i < half; i++) f[i] = pow((double)s.rope_base, -2.0 * i / dims) / (s.rope_factor > 0.0f ? (double)s.rope_factor : 1.0);
     if (s.yarn_factor > 0.0f) {
         const double factor = s.yarn_factor, two_pi = 6.283185307179586476925286766559;
         auto turn_dim = [&](double t) { return dims * log((double)s.yarn_original / (two_pi * t)) / (2.0 * log((double)s.rope_base)); };
@@ -328,10 +328,10 @@ static int ly_enqueue_route(b200_plan *p, bool decode, int n, const LyLayer &L, 
     if (decode) { // one row: the router's rows stream through the multi-CTA matvec, one warp selects
         if ((rc = ly_project<ly::EPI_STORE>(p, true, 1, x32, nullptr, L.w_router, nullptr, scores + extra, E, Y.ZR, nullptr, scores + extra, 0))) return rc;
         *nl += 2;
-        return launch_k(p, false, ly::k_moe_topk, dim3(1), dim3(32), (size_t)2 * scores * 4, (const float *)Y.ZR, scores, top, Y.moe_ids, Y.moe_wts, rm);
+        return launch_k(p, false, ly::k_moe_topk, dim3(1), dim3(32), (size_t)3 * scores * 4, (const float *)Y.ZR, scores, top, Y.moe_ids, Y.moe_wts, rm);
     }
     // a CTA per row: four warps share the row's experts
-    const size_t rsm = (size_t)(E + 2 * (scores + extra)) * 4;
+    const size_t rsm = (size_t)(E + 3 * (scores + extra)) * 4;
     ++*nl;
     if (!Y.f32) return launch_k(p, false, ly::k_moe_route<ly::bf16>, dim3(n), dim3(128), rsm, x16, (const ly::bf16 *)L.w_router, n, E, scores, top, 1, Y.moe_ids, Y.moe_wts, rm, extra, Y.SGL);
     return launch_k(p, false, ly::k_moe_route<float>, dim3(n), dim3(128), rsm, x32, (const ly::bf16 *)L.w_router, n, E, scores, top, 1, Y.moe_ids, Y.moe_wts, rm, extra, Y.SGL);

@@ -5,12 +5,13 @@
 //   * k_norm_rows       sandwich norm: x += N(y; w_post), optional pass prologue (x += x0, x += step), out = N(x; w_pre),
 //                       N(v; w) = v / sqrt(mean(v^2) + eps) * (w_off + w); also the embedding gather (x = scale * E[token], optionally
 //                       normalised); with post_plain the sublayer output is added as x += y * w_post (a layer scale behind a pre-norm);
+//                       the sublayer output may be a mixture of experts, assembled here from the chosen experts' rows and their weights;
 //   * k_matvec_bf16     decode projection: BF16 weight rows streamed with 128-bit loads, FP32 activation and accumulator,
 //                       bias or gated-activation epilogue (gelu_tanh(g) * u);
 //   * k_gemm_f32 / k_gemm_bf16   prefill projections for any M, N, K: true FP32 on the CUDA cores, or BF16 operands on the
 //                       tensor cores (mma.sync m16n8k16, FP32 accumulation), same epilogues;
-//   * k_qk_prep         whole-projection RMS norm of q and of k (one statistic over ALL heads), K / V rows into the window ring;
-//   * k_window_attention  sliding-window attention over a ring cache with a soft logit cap, a learned bucketed distance bias
+//   * k_qk_prep         whole-projection RMS norm of q and of k (one statistic over ALL heads), optional rotation, K / V rows into the window ring;
+//   * k_window_attention  sliding-window (or chunk-masked) attention over a ring cache with a soft logit cap, a learned bucketed distance bias
 //                       and a softmax whose denominator carries an extra exp(0) (a value-less sink), sigmoid output gate.
 // The projection kernels take optional operand VIEWS (MvView / GemmView): a row stride for A, per-head batches, grouped rows for a
 // mixture of experts, an input scale and a sigmoid-gate epilogue; the attention kernels take row strides for the key and value
@@ -26,13 +27,14 @@ namespace ly {
 typedef __nv_bfloat16 bf16;
 
 enum { EPI_STORE = 0, EPI_GATED = 1, EPI_ACT = 2 }; // C = A W^T (+ bias)  |  H = act(A Wg^T) * (A Wu^T), W = [Wg; Wu] stacked by rows  |  H = act(A W^T (+ bias))
-enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_RELU = 2, ACT_GELU_ERF = 3, ACT_RELU2 = 4 };
+enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_RELU = 2, ACT_GELU_ERF = 3, ACT_RELU2 = 4, ACT_NONE = 5 };
 
 __device__ __forceinline__ float bf_lo(unsigned v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf_hi(unsigned v) { return __uint_as_float(v & 0xffff0000u); }
 
 __device__ __forceinline__ float act_apply(int act, float z) {
     if (act == ACT_SILU) return z / (1.0f + expf(-z));
+    if (act == ACT_NONE) return z;
     if (act == ACT_RELU) return fmaxf(z, 0.0f);
     if (act == ACT_RELU2) { const float r = fmaxf(z, 0.0f); return r * r; }
     if (act == ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); // the exact GELU: z * Phi(z)
@@ -93,18 +95,39 @@ struct NormArgs {
     float w_off;         // added to every norm weight: 1 for weights stored as a deviation from one, 0 for weights used as stored
     int post_plain;      // 1: x += y * w_post (no statistic of y: a layer scale)
     const float *w_emb;  // [E] (nullable): the gathered embedding row is normalised, x = N(scale * emb[token]; w_emb)
+    float post_off;      // added to the weights of w_post (as w_off is to all others)
+    // sublayer output that is a mixture of experts (instead of y): sum over the `top` entries k of row r of wts[r * top + k] * (row of that entry in ys)
+    const float *ys;     // [entries][E] (nullable)
+    const int *ys_map;   // (nullable) entry e lives in row ys_map[e] of ys
+    const float *wts;
+    int top;
 };
+#define LY_NORM_TERMS 64 // entries of a mixture whose places and weights are kept in shared memory (more: read where they are)
 #define LY_NORM_THREADS 256
 
-__global__ void __launch_bounds__(LY_NORM_THREADS) k_norm_rows(NormArgs a) {
+// Out of a row without w_pre (out32 / out16 set): the row itself.  One CTA of NTH threads per row (a single wide row takes more threads: more of
+// its loads are in flight).  Dynamic shared memory: E floats, 2 * E with ys.
+template <int NTH>
+__global__ void __launch_bounds__(NTH) k_norm_rows(NormArgs a) {
     extern __shared__ __align__(16) float row[];
     __shared__ float red[32];
+    __shared__ size_t s_row[LY_NORM_TERMS];
+    __shared__ float s_wt[LY_NORM_TERMS];
     const int r = blockIdx.x, tid = threadIdx.x, E = a.E;
     const size_t src = (size_t)(a.gather ? a.gather[r] : r) * E, dst = (size_t)r * E;
+    const bool terms = a.ys && a.top <= LY_NORM_TERMS;
+    if (terms) {
+        if (tid < a.top) {
+            const size_t e = (size_t)r * a.top + tid;
+            s_row[tid] = (a.ys_map ? (size_t)a.ys_map[e] : e) * E;
+            s_wt[tid] = a.wts[e];
+        }
+        __syncthreads();
+    }
     if (a.emb) {
         const int token = a.tokens ? a.tokens[r] : a.st->token;
         const bf16 *e = a.emb + (size_t)token * E;
-        for (int i = tid; i < E; i += LY_NORM_THREADS) {
+        for (int i = tid; i < E; i += NTH) {
             const float v = __bfloat162float(e[i]) * a.emb_scale;
             row[i] = v;
             if (a.x0) a.x0[src + i] = v;
@@ -112,44 +135,73 @@ __global__ void __launch_bounds__(LY_NORM_THREADS) k_norm_rows(NormArgs a) {
         if (a.w_emb) {
             __syncthreads();
             float ss = 0.0f;
-            for (int i = tid; i < E; i += LY_NORM_THREADS) ss = fmaf(row[i], row[i], ss);
+            for (int i = tid; i < E; i += NTH) ss = fmaf(row[i], row[i], ss);
             ss = block_sum(ss, red);
             const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
-            for (int i = tid; i < E; i += LY_NORM_THREADS) {
+            for (int i = tid; i < E; i += NTH) {
                 const float v = row[i] * inv * (a.w_off + a.w_emb[i]);
                 row[i] = v;
                 if (a.x0) a.x0[src + i] = v;
             }
         }
     } else {
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] = a.x[src + i];
+        for (int i = tid; i < E; i += NTH) row[i] = a.x[src + i];
     }
     if (a.y && a.post_plain) {
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] = fmaf(a.y[src + i], a.w_post[i], row[i]);
+        for (int i = tid; i < E; i += NTH) row[i] = fmaf(a.y[src + i], a.w_post[i], row[i]);
+    } else if (a.ys) { // every thread touches its own entries of the assembled row only
+        float *yv = row + E, ss = 0.0f;
+        for (int i = tid; i < E; i += NTH) {
+            float s = 0.0f;
+            if (terms) {
+                for (int k0 = 0; k0 < a.top; k0 += 4) { // the loads of four entries are issued before the first is used
+                    float v[4];
+#pragma unroll
+                    for (int u = 0; u < 4; u++) v[u] = k0 + u < a.top ? __ldg(a.ys + s_row[k0 + u] + i) : 0.0f;
+#pragma unroll
+                    for (int u = 0; u < 4; u++) if (k0 + u < a.top) s = fmaf(s_wt[k0 + u], v[u], s);
+                }
+            } else {
+                for (int k = 0; k < a.top; k++) {
+                    const size_t e = (size_t)r * a.top + k;
+                    s = fmaf(a.wts[e], a.ys[(a.ys_map ? (size_t)a.ys_map[e] : e) * E + i], s);
+                }
+            }
+            yv[i] = s;
+            ss = fmaf(s, s, ss);
+        }
+        ss = block_sum(ss, red);
+        const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
+        for (int i = tid; i < E; i += NTH) row[i] += yv[i] * inv * (a.post_off + a.w_post[i]);
     } else if (a.y) {
         float ss = 0.0f;
-        for (int i = tid; i < E; i += LY_NORM_THREADS) { const float v = a.y[src + i]; ss = fmaf(v, v, ss); }
+        for (int i = tid; i < E; i += NTH) { const float v = a.y[src + i]; ss = fmaf(v, v, ss); }
         ss = block_sum(ss, red);
         const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] += a.y[src + i] * inv * (a.w_off + a.w_post[i]);
+        for (int i = tid; i < E; i += NTH) row[i] += a.y[src + i] * inv * (a.post_off + a.w_post[i]);
     }
     if (a.trace)
-        for (int i = tid; i < E; i += LY_NORM_THREADS) a.trace[src + i] = row[i];
+        for (int i = tid; i < E; i += NTH) a.trace[src + i] = row[i];
     if (a.add_x0)
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] += a.x0[src + i];
+        for (int i = tid; i < E; i += NTH) row[i] += a.x0[src + i];
     if (a.step)
-        for (int i = tid; i < E; i += LY_NORM_THREADS) row[i] += a.step[i];
-    if (!a.gather && (a.emb || a.y || a.add_x0 || a.step))
-        for (int i = tid; i < E; i += LY_NORM_THREADS) a.x[src + i] = row[i];
+        for (int i = tid; i < E; i += NTH) row[i] += a.step[i];
+    if (!a.gather && (a.emb || a.y || a.ys || a.add_x0 || a.step))
+        for (int i = tid; i < E; i += NTH) a.x[src + i] = row[i];
     if (a.w_pre) {
         float ss = 0.0f;
-        for (int i = tid; i < E; i += LY_NORM_THREADS) ss = fmaf(row[i], row[i], ss);
+        for (int i = tid; i < E; i += NTH) ss = fmaf(row[i], row[i], ss);
         ss = block_sum(ss, red);
         const float inv = 1.0f / sqrtf(ss / (float)E + a.eps);
-        for (int i = tid; i < E; i += LY_NORM_THREADS) {
+        for (int i = tid; i < E; i += NTH) {
             const float v = row[i] * inv * (a.w_off + a.w_pre[i]);
             if (a.out32) a.out32[dst + i] = v;
             if (a.out16) a.out16[dst + i] = __float2bfloat16_rn(v);
+        }
+    } else if (a.out32 || a.out16) {
+        for (int i = tid; i < E; i += NTH) {
+            if (a.out32) a.out32[dst + i] = row[i];
+            if (a.out16) a.out16[dst + i] = __float2bfloat16_rn(row[i]);
         }
     }
 }
@@ -178,6 +230,18 @@ __device__ __forceinline__ float dot_row_bf16(const bf16 *__restrict__ w, const 
     return warp_sum(acc);
 }
 
+// A row of a second token embedding as a factor: entry n of a result row is multiplied by table[token * ld + n].
+struct TokenGate {
+    const bf16 *table;     // (nullable) first column used of a [vocab][ld] table
+    int ld;
+    const int *tokens;     // [rows] (nullable: the step's own token)
+    const StepState *st;
+};
+__device__ __forceinline__ float token_gate(const TokenGate &g, int row, int n) {
+    const int token = g.tokens ? g.tokens[row] : g.st->token;
+    return __bfloat162float(g.table[(size_t)token * g.ld + n]);
+}
+
 // Optional second grid dimension of a decode projection: blockIdx.y = b selects a per-head operand (offsets b * w_bs / x_bs /
 // y_bs into W, x, y) and, with `group`, the weight matrix of expert group[b] (offset group[b] * w_gs).  in_scale[b] multiplies
 // the INPUT of a gated projection (act(s g) * (s u)); mul multiplies a stored result by sigmoid(mul[b * y_bs + n]).
@@ -188,6 +252,7 @@ struct MvView {
     const float *in_scale;
     const float *mul;
     int n_groups; // > 0: a CTA whose group[b] >= n_groups has nothing to do (an expert without weights: the identity)
+    TokenGate tg; // EPI_ACT: the activation is multiplied by the token's entry of a table
 };
 
 template <int EPI>
@@ -212,6 +277,7 @@ __global__ void __launch_bounds__(LY_MV_THREADS) k_matvec_bf16(const bf16 *__res
         } else if (EPI == EPI_ACT) {
             if (bias) v += bias[n];
             v = act_apply(act, v);
+            if (v_.tg.table) v *= token_gate(v_.tg, 0, n);
         } else {
             if (bias) v += bias[n];
             if (v_.mul) v *= 1.0f / (1.0f + expf(-v_.mul[(size_t)b * v_.y_bs + n]));
@@ -240,6 +306,7 @@ struct GemmView {
     const float *in_scale;
     const float *mul;
     int ldmul;
+    TokenGate tg; // EPI_ACT: the activation is multiplied by the entry of the row's token
 };
 
 // Fills the A / C row numbers of this CTA's 64 rows (-1: outside); returns false when the tile has no work.
@@ -270,7 +337,10 @@ __device__ __forceinline__ float gemm_epilogue(const GemmView &g, float a0, floa
         const float sc = g.in_scale ? g.in_scale[crow] : 1.0f;
         return act_apply(act, a0 * sc) * (a1 * sc);
     }
-    if (EPI == EPI_ACT) return act_apply(act, a0 + (bias ? bias[n] : 0.0f));
+    if (EPI == EPI_ACT) {
+        const float h = act_apply(act, a0 + (bias ? bias[n] : 0.0f));
+        return g.tg.table ? h * token_gate(g.tg, crow, n) : h;
+    }
     float v = a0 + (bias ? bias[n] : 0.0f);
     if (g.mul) v *= 1.0f / (1.0f + expf(-g.mul[(size_t)crow * g.ldmul + c_off + n]));
     return v;
@@ -478,7 +548,21 @@ struct WindowAttn {
     int maps;                    // > 1: every head carries `maps` score maps over the same values.  `heads` then counts (head, map) pairs, pair
                                  // p = head * maps + map reads key slice (value head) * maps + map of a key row [kv_heads][maps][dk] and the
                                  // values of its head; the output keeps one row of dv entries per pair
+    int chunked;                 // 1: position i sees j <= i with i / window == j / window (chunks counted from position 0) instead of the last `window`
+    float out_scale = 1.0f;      // multiplies the (gated) output
+    // k_qk_prep: rotation of the first rope_dims entries of every query and key head behind the whole-projection norm (0: none)
+    const float *cs;             // [position][rope_dims / 2][2] = (cos, sin)
+    int rope_dims, rope_layout;
 };
+// First position that `pos` sees
+__device__ __forceinline__ int window_first(const WindowAttn &a, int pos) {
+    if (a.chunked) return pos / a.window * a.window;
+    return pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
+}
+__device__ __forceinline__ void rope_pair_index(int i, int dims, int layout, int &u, int &v) {
+    if (layout) { u = 2 * i; v = 2 * i + 1; }
+    else { u = i; v = i + dims / 2; }
+}
 // Row layout of the fused projection output: [q: heads*dk | k: kv_heads*dk | v: kv_heads*dv | g: heads*dv]
 
 // One CTA per row: projection biases, RMS statistics over the WHOLE q and the WHOLE k projection, q normalised in place,
@@ -507,15 +591,44 @@ __global__ void __launch_bounds__(256) k_qk_prep(float *__restrict__ P, int ldp,
         ss = block_sum(ss, red);
         kinv = 1.0f / sqrtf(ss / (float)kd + a.eps);
     }
+    for (int i = tid; i < vd; i += 256) {
+        vc[(size_t)slot * vd + i] = v[i];
+        if (vc16) vc16[(size_t)slot * vd + i] = __float2bfloat16_rn(v[i]);
+    }
+    if (a.rope_dims > 0) { // q heads, then k heads: rotated pairs, then the entries behind them
+        const int half = a.rope_dims / 2, rest = a.dk - a.rope_dims;
+        const float *cs = a.cs + (size_t)(st->pos + r) * half * 2;
+        auto emit = [&](int hd, int i, float x) {
+            if (hd < a.heads) { q[hd * a.dk + i] = x; return; }
+            const size_t at = (size_t)slot * kd + (size_t)(hd - a.heads) * a.dk + i;
+            kc[at] = x;
+            if (kc16) kc16[at] = __float2bfloat16_rn(x);
+        };
+        auto normed = [&](int hd, int i) { // q and k lie side by side in the row
+            const int at = hd * a.dk + i;
+            const float x = q[at];
+            if (hd < a.heads) return a.qnorm ? x * qinv * a.qnorm[at] : x;
+            return a.knorm ? x * kinv * a.knorm[at - qd] : x;
+        };
+        for (int e = tid; e < (a.heads + a.kv_heads) * half; e += 256) {
+            const int hd = e / half, i = e % half;
+            int u, w;
+            rope_pair_index(i, a.rope_dims, a.rope_layout, u, w);
+            const float xu = normed(hd, u), xw = normed(hd, w), co = cs[2 * i], si = cs[2 * i + 1];
+            emit(hd, u, fmaf(xu, co, -(xw * si)));
+            emit(hd, w, fmaf(xw, co, xu * si));
+        }
+        for (int e = tid; e < (a.heads + a.kv_heads) * rest; e += 256) {
+            const int hd = e / rest, i = a.rope_dims + e % rest;
+            emit(hd, i, normed(hd, i));
+        }
+        return;
+    }
     for (int i = tid; i < qd; i += 256) q[i] = a.qnorm ? q[i] * qinv * a.qnorm[i] : q[i];
     for (int i = tid; i < kd; i += 256) {
         const float kv = a.knorm ? k[i] * kinv * a.knorm[i] : k[i];
         kc[(size_t)slot * kd + i] = kv;
         if (kc16) kc16[(size_t)slot * kd + i] = __float2bfloat16_rn(kv); // BF16 twin row for the tensor-core prefill attention
-    }
-    for (int i = tid; i < vd; i += 256) {
-        vc[(size_t)slot * vd + i] = v[i];
-        if (vc16) vc16[(size_t)slot * vd + i] = __float2bfloat16_rn(v[i]);
     }
 }
 
@@ -547,7 +660,7 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
     const int gk = a.maps > 1 ? g * a.maps + h % a.maps : a.k_heads > 0 ? h / (a.heads / a.k_heads) : g;
     const float sink_v = a.sink_logit ? a.sink_logit[h] : 0.0f;
     const int pos = st->pos + r;
-    int lo = pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
+    int lo = window_first(a, pos);
     int nk = pos - lo + 1;
     if (splits > 1) { // this CTA's share of the window; everything below indexes keys as lo + j, j < nk
         const int chunk = (nk + splits - 1) / splits, jb = z * chunk;
@@ -655,7 +768,7 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
                 if (splits > 1) { my_o[d + e] = o; continue; }
                 o *= inv;
                 if (a.gate) o *= 1.0f / (1.0f + expf(-gate[(d + e) * gs]));
-                store_out<OUT_T>(out + (size_t)r * ldo + (size_t)h * a.dv + d + e, o);
+                store_out<OUT_T>(out + (size_t)r * ldo + (size_t)h * a.dv + d + e, o * a.out_scale);
             }
         }
     }
@@ -683,7 +796,7 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
         }
         o /= Lsum;
         if (a.gate) o *= 1.0f / (1.0f + expf(-gate[d * gs]));
-        store_out<OUT_T>(out + (size_t)r * ldo + (size_t)h * a.dv + d, o);
+        store_out<OUT_T>(out + (size_t)r * ldo + (size_t)h * a.dv + d, o * a.out_scale);
     }
     if (tid == 0) ks_.count[cell] = 0u; // ready for the next launch
 }
@@ -737,7 +850,7 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
     const int pos0 = st->pos;
     const int rows = n - r0 < BM ? n - r0 : BM;
     const int q_lo = pos0 + r0, q_hi = pos0 + r0 + rows - 1;
-    const int k_lo = q_lo - a.window + 1 > 0 ? q_lo - a.window + 1 : 0;
+    const int k_lo = window_first(a, q_lo);
     auto load_tile = [&](int buf, int kt0) {
         bf16(*Kd)[DK + 8] = reinterpret_cast<bf16(*)[DK + 8]>(smraw + QT + buf * KT);
         bf16(*Vd)[DV + 8] = reinterpret_cast<bf16(*)[DV + 8]>(smraw + QT + 2 * KT + buf * VT);
@@ -794,6 +907,8 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
     const int prow[2] = {pos0 + r0 + warp * 16 + g, pos0 + r0 + warp * 16 + g + 8}; // positions of this thread's two rows
     const bool vrow[2] = {warp * 16 + g < rows, warp * 16 + g + 8 < rows};
     const int w_lo = pos0 + r0 + warp * 16, w_hi = w_lo + 15; // positions of this warp's rows
+    const int w_first = window_first(a, w_lo);                // first key any of them sees
+    const int c_first[2] = {a.chunked ? window_first(a, prow[0]) : 0, a.chunked ? window_first(a, prow[1]) : 0};
     const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
     int buf = 0;
     for (int kt0 = k_lo; kt0 <= q_hi; kt0 += 64, buf ^= 1) {
@@ -803,7 +918,7 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
         } else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         // a warp whose rows see no key of this tile (all later, or all beyond the window) skips the arithmetic
-        if (kt0 <= w_hi && kt0 + 63 > w_lo - a.window) {
+        if (kt0 <= w_hi && kt0 + 63 >= w_first) {
             bf16(*Ks)[DK + 8] = reinterpret_cast<bf16(*)[DK + 8]>(smraw + QT + buf * KT);
             bf16(*Vs)[DV + 8] = reinterpret_cast<bf16(*)[DV + 8]>(smraw + QT + 2 * KT + buf * VT);
             // S = Q K^T for this warp's 16 rows x 64 keys
@@ -829,7 +944,7 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
                     const int rr = e >> 1, pj = kt0 + j * 8 + 2 * t + (e & 1), dist = prow[rr] - pj;
                     float v = sc[j][e] * a.scale;
                     if (a.softcap > 0.0f) v = a.softcap * tanh_fast(v * inv_cap);
-                    if (vrow[rr] && dist >= 0 && dist < a.window) v += sbias[dist];
+                    if (vrow[rr] && dist >= 0 && dist < a.window && pj >= c_first[rr]) v += sbias[dist];
                     else v = -INFINITY;
                     sc[j][e] = v;
                     tmax[rr] = fmaxf(tmax[rr], v);
@@ -887,7 +1002,7 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
     for (int rr = 0; rr < 2; rr++) {
         if (!vrow[rr]) continue;
         const int r = r0 + warp * 16 + g + rr * 8;
-        const float inv = lrow[rr] > 0.0f ? 1.0f / lrow[rr] : 0.0f;
+        const float inv = lrow[rr] > 0.0f ? a.out_scale / lrow[rr] : 0.0f;
         const float *gate = (a.gate_src ? a.gate_src + (size_t)r * a.gate_ld : P + (size_t)r * ldp) + (a.gate_off >= 0 ? a.gate_off : qd + kd + vd) +
                             (a.gate_heads ? (size_t)h : (size_t)h * DV);
         const float ghead = a.gate && a.gate_heads ? 1.0f / (1.0f + expf(-gate[0])) : 1.0f;

@@ -21,13 +21,16 @@
 // experts reading two norms of the same residual row).  Sandwich and pre-norm layers choose their mixer per layer: windowed
 // attention (optionally with rotation, values taken from the keys, head temperatures and head-mixed scores: k_rope_mix_prep
 // replaces k_qk_prep) or the gated delta rule (k_delta_prep -> k_delta_rule -> k_head_norm_gate), whose recurrent state and
-// convolution inputs live per RUN next to the rings.  Two further block kinds: outnorm_plan.cuh, layernorm_plan.cuh.
+// convolution inputs live per RUN next to the rings.  Two further block kinds: outnorm_plan.cuh, layernorm_plan.cuh; further mixers and
+// feed-forwards of the sandwich block and the per-layer token input: sandwich_plan.cuh.
 #pragma once
 #include "layered.cuh"
 #include "latent.cuh"
 #include "delta.cuh"
 #include "recurrent.cuh"
 #include "mlstm.cuh"
+#include "selective.cuh"
+#include "lightning.cuh"
 
 struct LyLayer {
     b200_layer_spec s{};
@@ -82,6 +85,18 @@ struct LyLayer {
     ly::bf16 *w_sgu = nullptr, *w_sdown = nullptr;
     CUtensorMap m_sgate, m_sup, m_sdown, m_sh;
     bool tc_sgu = false, tc_sdown = false;
+    // lightning: decays per head.  Attention + scan: ad = the attention's output columns (gd = ad + scan_inner), x_off = first scan column of a projection
+    // row ([x | z]), W_x with nx rows (nxp with padding), W_dt, decay exponents; conv_w, conv_b, dt_bias, ssd_d as above
+    float *decay = nullptr, *a2 = nullptr;
+    int ad = 0, x_off = 0, nx = 0, nxp = 0;
+    ly::bf16 *w_x = nullptr, *w_dt = nullptr;
+    CUtensorMap m_wx, m_u, m_wdt, m_dt16;
+    bool tc_wx = false, tc_wdt = false;
+    // per-layer token input
+    ly::bf16 *w_sgate = nullptr, *w_sproj = nullptr;
+    float *side_norm = nullptr;
+    CUtensorMap m_tsg, m_tsp;
+    bool tc_side = false;
 };
 struct LyRun {
     int layer = 0, pass = -1;
@@ -152,6 +167,18 @@ struct Layered {
     ly::bf16 *bigram = nullptr;
     int *tok_hist = nullptr;
     double *pos_freq = nullptr;
+    // attention + scan: parameter rows [r | B | C] of the scan, BF16 r; the branch stream and its fork / join events
+    float *XP = nullptr;
+    ly::bf16 *DT16 = nullptr;
+    int maxX = 0, maxRank = 0;
+    CUtensorMap m_xp_c, m_dt_c;
+    cudaStream_t branch = nullptr;
+    cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
+    // per-layer token input: second embedding table [vocab][layers * side_dim], gated rows
+    ly::bf16 *side_emb = nullptr, *SIDE16 = nullptr;
+    float *SIDE32 = nullptr;
+    int side_pad = 0;
+    CUtensorMap m_side;
 };
 
 // What ly_project needs to take the tcgen05 route: operand and result descriptors (nullptr = CUDA-core / mma.sync kernels).
@@ -217,6 +244,11 @@ static int ly_bucket(int n, int rows, double far) {
 }
 
 static void ly_free(b200_plan *p) {
+    if (p->ly) {
+        if (p->ly->ev_fork) cudaEventDestroy(p->ly->ev_fork);
+        if (p->ly->ev_join) cudaEventDestroy(p->ly->ev_join);
+        if (p->ly->branch) cudaStreamDestroy(p->ly->branch);
+    }
     delete p->ly;
     p->ly = nullptr;
 }
@@ -228,13 +260,13 @@ static size_t ly_att_smem(const b200_layer_spec &s, int ring) {
     return ly_att_smem(s.mixer == B200_MIXER_LATENT_ATTENTION ? s.kv_rank + s.rot_dim : s.head_mix ? s.kv_heads * s.key_dim : s.key_dim, s.window);
 }
 
-// Instances of the tensor-core prefill attention: (key size, value size) = (64, 64), (128, 128), (192, 128); 0 = none.
+// Instances of the tensor-core prefill attention: (key size, value size) = (64, 64), (128, 128), (192, 128), (128, 64), (256, 128), (64, 32); 0 = none.
 static int ly_mma_kind(int dk, int dv) {
-    return dk == 64 && dv == 64 ? 1 : dk == 128 && dv == 128 ? 2 : dk == 192 && dv == 128 ? 3 : dk == 128 && dv == 64 ? 4 : dk == 256 && dv == 128 ? 5 : 0;
+    return dk == 64 && dv == 64 ? 1 : dk == 128 && dv == 128 ? 2 : dk == 192 && dv == 128 ? 3 : dk == 128 && dv == 64 ? 4 : dk == 256 && dv == 128 ? 5 : dk == 64 && dv == 32 ? 6 : 0;
 }
 static size_t ly_mma_smem(int kind, int window) {
     return kind == 1 ? ly::att_mma_smem_bytes<64, 64>(window) : kind == 2 ? ly::att_mma_smem_bytes<128, 128>(window) : kind == 3 ? ly::att_mma_smem_bytes<192, 128>(window)
-         : kind == 4 ? ly::att_mma_smem_bytes<128, 64>(window) : ly::att_mma_smem_bytes<256, 128>(window);
+         : kind == 4 ? ly::att_mma_smem_bytes<128, 64>(window) : kind == 5 ? ly::att_mma_smem_bytes<256, 128>(window) : ly::att_mma_smem_bytes<64, 32>(window);
 }
 static int ly_launch_mma(b200_plan *p, int kind, int n, int heads, int window, const float *P, int ldp, const ly::WindowAttn &wa, const ly::bf16 *k16, const ly::bf16 *v16,
                          const StepState *st, ly::bf16 *out, int ldo, float *out32 = nullptr) {
@@ -244,6 +276,7 @@ static int ly_launch_mma(b200_plan *p, int kind, int n, int heads, int window, c
     if (kind == 2) return launch_k(p, false, ly::k_window_attention_mma<128, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
     if (kind == 4) return launch_k(p, false, ly::k_window_attention_mma<128, 64>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
     if (kind == 5) return launch_k(p, false, ly::k_window_attention_mma<256, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
+    if (kind == 6) return launch_k(p, false, ly::k_window_attention_mma<64, 32>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
     return launch_k(p, false, ly::k_window_attention_mma<192, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
 }
 
@@ -256,6 +289,8 @@ static ly::WindowAttn ly_attn_args(const Layered &Y, const LyLayer &L) {
     a.rel = L.rel; a.bucket = L.bucket; a.qnorm = L.qnorm; a.knorm = L.knorm;
     a.sink = L.s.sink; a.gate = L.s.gate; a.gate_off = L.qd + L.kd + L.pv; a.eps = Y.c.norm_eps;
     a.sink_logit = L.sink_logit; a.gate_heads = L.s.gate == 2;
+    a.chunked = L.s.mask_chunked;
+    if (L.s.mixer == B200_MIXER_ATTENTION_SCAN) { a.cs = L.rope; a.rope_dims = L.s.rope_dims; a.rope_layout = L.s.rope_layout; a.out_scale = L.s.branch_scale[0]; }
     if (L.mixprep) { // the query comes from k_rope_mix_prep's buffer (temperature and head mixing folded in), the gate from the projection row
         a.dk = L.dk_eff; a.k_heads = L.k_heads; a.qnorm = a.knorm = nullptr;
         a.gate_src = Y.PROJ; a.gate_ld = Y.maxP;
@@ -304,9 +339,47 @@ static int ly_project(b200_plan *p, bool decode, int n, const float *a32, const 
     return launch_k(p, false, ly::k_gemm_bf16<EPI, float>, grid, dim3(128), (size_t)0, a16, W, bias, c32, n, N, K, ldc, act, ly::GemmView{});
 }
 
+// Attention of one layer with its own rings, from the projection rows in PROJ to the (gated) heads in ATT32 / ATT16 (row stride L.gd).
+static int ly_enqueue_attention(b200_plan *p, bool decode, int n, const StepState *st, const LyRun &R, const LyLayer &L, int *nl) {
+    Layered &Y = *p->ly;
+    const bool h16 = !decode && !Y.f32;
+    int rc;
+    const ly::WindowAttn wa = ly_attn_args(Y, L);
+    const float *qsrc = Y.PROJ; // where the attention kernels read the query rows
+    int ldq = Y.maxP;
+    if (L.mixprep) {
+        ly::RopeMixArgs ra{};
+        ra.heads = L.s.heads; ra.kv_heads = L.s.kv_heads; ra.dk = L.s.key_dim; ra.dv = L.s.value_dim; ra.rope_dims = L.s.rope_dims; ra.rope_layout = L.s.rope_layout;
+        ra.cs = L.rope; ra.temp = L.temp; ra.talk = L.talk; ra.value_from_key = L.s.value_from_key; ra.ring = Y.ring;
+        qsrc = Y.Q; ldq = L.s.heads * L.dk_eff;
+        const int hpc = decode ? 1 : ROPE_MIX_HEADS; // one row: a CTA per head; a chunk: several heads share the rotation of the row
+        rc = launch_k(p, false, ly::k_rope_mix_prep, dim3(n, (L.s.heads + hpc - 1) / hpc + 1), dim3(ROPE_MIX_THREADS), (size_t)(L.qd > L.kd ? L.qd : L.kd) * 4, (const float *)Y.PROJ, Y.maxP, ra,
+                      (const float *)L.b_proj, Y.Q, ldq, R.kc, R.vc, R.kc16, R.vc16, st, hpc);
+    } else
+        rc = launch_k(p, false, ly::k_qk_prep, dim3(n), dim3(256), (size_t)0, Y.PROJ, Y.maxP, wa, (const float *)L.b_proj, R.kc, R.vc, R.kc16, R.vc16, st);
+    if (rc) return rc;
+    ++*nl;
+    const size_t asm_ = ly_att_smem(L.s, Y.ring);
+    const int mma = ly_mma_kind(L.mixprep ? L.dk_eff : L.s.key_dim, L.s.value_dim);
+    if (h16 && R.kc16 && mma)
+        rc = ly_launch_mma(p, mma, n, L.s.heads, L.s.window, qsrc, ldq, wa, (const ly::bf16 *)R.kc16, (const ly::bf16 *)R.vc16, st, Y.ATT16, L.gd);
+    else if (h16) rc = launch_k(p, false, ly::k_window_attention<ly::bf16>, dim3(n, L.s.heads), dim3(LY_ATT_THREADS), asm_, qsrc, ldq, wa,
+                           (const float *)R.kc, (const float *)R.vc, st, Y.ATT16, L.gd, ly::KeySplit{nullptr, nullptr, nullptr});
+    else {
+        // the decode step has one row and few heads: split every head's window over several CTAs so that the SMs are used
+        int sp = 1;
+        if (decode && Y.split.o && L.s.window >= 64) { sp = p->n_sms / L.s.heads; if (sp > Y.max_splits) sp = Y.max_splits; if (sp < 1) sp = 1; }
+        rc = launch_k(p, false, ly::k_window_attention<float>, dim3(n, L.s.heads, sp), dim3(LY_ATT_THREADS), asm_, qsrc, ldq, wa,
+                      (const float *)R.kc, (const float *)R.vc, st, Y.ATT32, L.gd, sp > 1 ? Y.split : ly::KeySplit{nullptr, nullptr, nullptr});
+    }
+    ++*nl;
+    return rc;
+}
+
 #include "latent_plan.cuh"
 #include "outnorm_plan.cuh"
 #include "layernorm_plan.cuh"
+#include "sandwich_plan.cuh"
 
 // Enqueue the forward of n rows on p->stream.  decode: the single-token step (row 0, position and token from *st).
 // with_head (decode only): final norm + classifier into p->logits.  Prefill leaves the finished residual rows in X.
@@ -318,20 +391,26 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
     const int E = Y.c.width;
     const bool h16 = !decode && !Y.f32; // prefill in BF16 mode rounds GEMM operands to BF16
     int nl = 0, rc;
-    const float *pend_y = nullptr, *pend_w = nullptr;
+    const float *pend_y = nullptr, *pend_w = nullptr, *pend_ys = nullptr; // pend_ys: a mixture of experts, assembled by the next row kernel
+    const int *pend_map = nullptr;
+    int pend_top = 0;
+    float pend_off = Y.w_off;
     float *pend_trace = nullptr;
-    auto norm = [&](bool embed, bool add_x0, const float *step, const float *w_pre) {
+    auto norm = [&](bool embed, bool add_x0, const float *step, const float *w_pre, bool raw = false) { // raw: the residual row itself as a BF16 operand
         ly::NormArgs a{};
         a.x = Y.X; a.x0 = Y.has_loop && !Y.prenorm ? Y.X0 : nullptr;
-        a.y = pend_y; a.w_post = pend_w;
+        a.y = pend_y; a.w_post = pend_w; a.post_off = pend_off;
+        a.ys = pend_ys; a.ys_map = pend_map; a.wts = Y.moe_wts; a.top = pend_top;
         a.w_off = Y.w_off; a.post_plain = Y.prenorm ? 1 : 0; a.w_emb = embed ? Y.emb_norm : nullptr;
         a.emb = embed ? Y.emb : nullptr; a.tokens = tokens; a.st = st; a.emb_scale = Y.c.embedding_scale;
         a.add_x0 = add_x0 ? 1 : 0; a.step = step; a.w_pre = w_pre;
-        a.out32 = w_pre && !h16 ? Y.A32 : nullptr; a.out16 = w_pre && h16 ? Y.A16 : nullptr;
+        a.out32 = w_pre && !h16 ? Y.A32 : nullptr; a.out16 = (w_pre || raw) && h16 ? Y.A16 : nullptr;
         a.gather = nullptr; a.trace = pend_trace; a.eps = Y.c.norm_eps; a.E = E;
-        pend_y = pend_w = nullptr; pend_trace = nullptr;
+        const size_t sm = (size_t)(pend_ys ? 2 : 1) * E * 4;
+        pend_y = pend_w = pend_ys = nullptr; pend_map = nullptr; pend_top = 0; pend_off = Y.w_off; pend_trace = nullptr;
         nl++;
-        return launch_k(p, false, ly::k_norm_rows, dim3(n), dim3(LY_NORM_THREADS), (size_t)E * 4, a);
+        if (n == 1 && E >= 2048) return launch_k(p, false, ly::k_norm_rows<1024>, dim3(1), dim3(1024), sm, a);
+        return launch_k(p, false, ly::k_norm_rows<LY_NORM_THREADS>, dim3(n), dim3(LY_NORM_THREADS), sm, a);
     };
     for (size_t r = 0; r < Y.runs.size(); r++) {
         const LyRun &R = Y.runs[r];
@@ -371,38 +450,13 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
             if ((rc = launch_k(p, false, ly::k_head_norm_gate, dim3(n), dim3(256), (size_t)0, (const float *)Y.DO, Y.maxDO, (const float *)(Y.PROJ + L.dC + 2 * L.s.heads), Y.maxP, ha,
                                h16 ? (float *)nullptr : Y.ATT32, h16 ? Y.ATT16 : (ly::bf16 *)nullptr, L.gd))) return rc;
             nl += 3;
+        } else if (L.s.mixer == B200_MIXER_LIGHTNING) {
+            if ((rc = ly_enqueue_lightning(p, decode, n, st, R, L, &nl))) return rc;
+        } else if (L.s.mixer == B200_MIXER_ATTENTION_SCAN) {
+            if ((rc = ly_enqueue_attention_scan(p, decode, n, st, R, L, &nl))) return rc;
         } else {
-        const ly::WindowAttn wa = ly_attn_args(Y, L);
-        const float *qsrc = Y.PROJ; // where the attention kernels read the query rows
-        int ldq = Y.maxP;
-        if (L.mixprep) {
-            ly::RopeMixArgs ra{};
-            ra.heads = L.s.heads; ra.kv_heads = L.s.kv_heads; ra.dk = L.s.key_dim; ra.dv = L.s.value_dim; ra.rope_dims = L.s.rope_dims; ra.rope_layout = L.s.rope_layout;
-            ra.cs = L.rope; ra.temp = L.temp; ra.talk = L.talk; ra.value_from_key = L.s.value_from_key; ra.ring = Y.ring;
-            qsrc = Y.Q; ldq = L.s.heads * L.dk_eff;
-            const int hpc = decode ? 1 : ROPE_MIX_HEADS; // one row: a CTA per head; a chunk: several heads share the rotation of the row
-            rc = launch_k(p, false, ly::k_rope_mix_prep, dim3(n, (L.s.heads + hpc - 1) / hpc + 1), dim3(ROPE_MIX_THREADS), (size_t)(L.qd > L.kd ? L.qd : L.kd) * 4, (const float *)Y.PROJ, Y.maxP, ra,
-                          (const float *)L.b_proj, Y.Q, ldq, R.kc, R.vc, R.kc16, R.vc16, st, hpc);
-        } else
-            rc = launch_k(p, false, ly::k_qk_prep, dim3(n), dim3(256), (size_t)0, Y.PROJ, Y.maxP, wa, (const float *)L.b_proj, R.kc, R.vc, R.kc16, R.vc16, st);
-        if (rc) return rc;
-        nl++;
-        const size_t asm_ = ly_att_smem(L.s, Y.ring);
-        const int mma = ly_mma_kind(L.mixprep ? L.dk_eff : L.s.key_dim, L.s.value_dim);
-        if (h16 && R.kc16 && mma)
-            rc = ly_launch_mma(p, mma, n, L.s.heads, L.s.window, qsrc, ldq, wa, (const ly::bf16 *)R.kc16, (const ly::bf16 *)R.vc16, st, Y.ATT16, L.gd);
-        else if (h16) rc = launch_k(p, false, ly::k_window_attention<ly::bf16>, dim3(n, L.s.heads), dim3(LY_ATT_THREADS), asm_, qsrc, ldq, wa,
-                               (const float *)R.kc, (const float *)R.vc, st, Y.ATT16, L.gd, ly::KeySplit{nullptr, nullptr, nullptr});
-        else {
-            // the decode step has one row and few heads: split every head's window over several CTAs so that the SMs are used
-            int sp = 1;
-            if (decode && Y.split.o && L.s.window >= 64) { sp = p->n_sms / L.s.heads; if (sp > Y.max_splits) sp = Y.max_splits; if (sp < 1) sp = 1; }
-            rc = launch_k(p, false, ly::k_window_attention<float>, dim3(n, L.s.heads, sp), dim3(LY_ATT_THREADS), asm_, qsrc, ldq, wa,
-                          (const float *)R.kc, (const float *)R.vc, st, Y.ATT32, L.gd, sp > 1 ? Y.split : ly::KeySplit{nullptr, nullptr, nullptr});
+            if ((rc = ly_enqueue_attention(p, decode, n, st, R, L, &nl))) return rc;
         }
-        if (rc) return rc;
-        nl++;
-        } // windowed attention
         if ((rc = ly_project<ly::EPI_STORE>(p, decode, n, Y.ATT32, Y.ATT16, L.w_o, nullptr, E, L.gd, Y.Y, nullptr, E, 0, &t_o))) return rc;
         nl++;
         pend_y = Y.Y; pend_w = Y.prenorm ? L.ls1 : L.norm1b;
@@ -414,6 +468,21 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
             if ((rc = ly_project<ly::EPI_STORE>(p, decode, n, Y.H32, Y.H16, L.w_down, nullptr, E, F, Y.Y, nullptr, E, 0, &t_down))) return rc;
             nl++;
             pend_y = Y.Y; pend_w = Y.prenorm ? L.ls2 : L.norm2b;
+        } else if (L.s.ff_kind == B200_FF_DENSE_PLAIN) {
+            if ((rc = norm(false, false, nullptr, L.norm2))) return rc;
+            if ((rc = ly_enqueue_plain_ff(p, decode, n, L, &nl))) return rc;
+            pend_y = Y.Y; pend_w = L.norm2b;
+        } else if (L.s.ff_kind == B200_FF_MOE) {
+            if ((rc = norm(false, false, nullptr, L.norm2))) return rc;
+            const ly::RouteMode rm{3, nullptr, L.s.ff_experts, 1.0f, nullptr, L.s.moe_groups, L.s.moe_keep};
+            if ((rc = ly_enqueue_route(p, decode, n, L, Y.A32, Y.A16, L.s.ff_experts, 0, rm, &nl))) return rc;
+            if ((rc = ly_enqueue_experts(p, decode, n, L, Y.A32, Y.A16, L.s.ff_experts, false, &pend_ys, &pend_map, &nl))) return rc;
+            pend_top = L.s.ff_top; pend_w = L.norm2b;
+        }
+        if (Y.c.side_dim > 0) {
+            if ((rc = norm(false, false, nullptr, nullptr, true))) return rc;
+            if ((rc = ly_enqueue_side(p, decode, n, st, tokens, R.layer, L, &nl))) return rc;
+            pend_y = Y.Y; pend_w = L.side_norm; pend_off = 0.0f;
         }
         pend_trace = trace ? trace + r * (size_t)Y.cap * E : nullptr;
     }
@@ -496,6 +565,7 @@ static int ly_tc_init(b200_plan *p) {
                        pg::make_map(&L.m_moe_down, L.w_down, X * E, F, pg::BN) == 0 && pg::make_map(&L.m_moe_h, Y.HS16, (uint64_t)Y.max_tiles128 * 128, F, pg::BM) == 0;
         }
     if (Y.outnorm) ly_outnorm_tc_init(p);
+    if (Y.c.block == B200_BLOCK_SANDWICH) ly_sandwich_tc_init(p);
     for (LyLayer &L : Y.layers) { // queries out of a query latent
         const int N = L.s.heads * L.s.key_dim, Rq = L.s.q_rank;
         if (L.s.mixer == B200_MIXER_LATENT_ATTENTION && Rq > 0)
@@ -512,7 +582,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     Layered &Y = *Yp;
     Y.c = *cfg;
     const b200_layered_config &c = Y.c;
-    if (c.arch != B200_ARCH_PIBIDRA && c.arch != B200_ARCH_LATUSUN && c.arch != B200_ARCH_LEROSUN && c.arch != B200_ARCH_DINUZEN && c.arch != B200_ARCH_KEGASUN) return fail(p, B200_ERR_UNSUPPORTED, "unknown layered arch %d", c.arch);
+    if (c.arch != B200_ARCH_PIBIDRA && c.arch != B200_ARCH_LATUSUN && c.arch != B200_ARCH_LEROSUN && c.arch != B200_ARCH_DINUZEN && c.arch != B200_ARCH_KEGASUN && c.arch != B200_ARCH_ZULESUN) return fail(p, B200_ERR_UNSUPPORTED, "unknown layered arch %d", c.arch);
     if (c.block != B200_BLOCK_SANDWICH && c.block != B200_BLOCK_PARALLEL && c.block != B200_BLOCK_PRENORM && c.block != B200_BLOCK_OUTNORM && c.block != B200_BLOCK_LAYERNORM) return fail(p, B200_ERR_BAD_ARG, "unknown block kind %d", c.block);
     Y.outnorm = c.block == B200_BLOCK_OUTNORM;
     const bool outn = Y.outnorm;
@@ -526,6 +596,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     const bool par = c.block == B200_BLOCK_PARALLEL, lnb = c.block == B200_BLOCK_LAYERNORM;
     if (lnb && c.loop_times >= 0 && c.loop_stop > c.loop_start) return fail(p, B200_ERR_UNSUPPORTED, "layer-norm blocks do not loop");
     if (lnb && (c.bigram_buckets < 0 || (c.sinusoid && !(c.sinusoid_base > 0.0f)))) return fail(p, B200_ERR_BAD_ARG, "%d bigram buckets, sinusoid base %g", c.bigram_buckets, (double)c.sinusoid_base);
+    if (c.side_dim < 0 || (c.side_dim > 0 && c.block != B200_BLOCK_SANDWICH)) return fail(p, B200_ERR_UNSUPPORTED, "per-layer token input of %d entries in block kind %d", c.side_dim, c.block);
     if (par && Y.has_loop && c.loop_stop > c.loop_start) return fail(p, B200_ERR_UNSUPPORTED, "parallel blocks do not loop");
     if (c.width <= 0 || c.vocab_size <= 0 || c.n_layers <= 0 || c.context_length <= 0) return fail(p, B200_ERR_BAD_ARG, "width, vocabulary, layers and context must be positive");
     if (c.compute != B200_COMPUTE_BF16 && c.compute != B200_COMPUTE_F32) return fail(p, B200_ERR_BAD_ARG, "compute must be B200_COMPUTE_BF16 or B200_COMPUTE_F32");
@@ -583,11 +654,16 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             ly_latent_buffers(Y, L);
             continue;
         }
+        if (c.block == B200_BLOCK_SANDWICH && (rc = ly_sandwich_ff_sizes(p, l, s))) return rc;
+        if (c.block == B200_BLOCK_SANDWICH && (s.mixer == B200_MIXER_LIGHTNING || s.mixer == B200_MIXER_ATTENTION_SCAN)) {
+            if ((rc = ly_sandwich_mixer_sizes(p, l, L))) return rc;
+            continue;
+        }
         if (s.mixer != B200_MIXER_WINDOW_ATTENTION && s.mixer != B200_MIXER_GATED_DELTA) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: mixer %d", l, s.mixer);
         if (s.mixer == B200_MIXER_GATED_DELTA) L.s.window = 1; // a recurrent state, no ring
         if (s.heads <= 0 || s.kv_heads <= 0 || s.heads % s.kv_heads || s.key_dim <= 0 || s.value_dim <= 0 || s.window <= 0)
             return fail(p, B200_ERR_BAD_ARG, "layer %d: heads %d / kv heads %d / key %d / value %d / window %d", l, s.heads, s.kv_heads, s.key_dim, s.value_dim, s.window);
-        if (s.ff_kind != B200_FF_NONE && s.ff_kind != B200_FF_DENSE_GATED) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", l, s.ff_kind);
+        if (c.block != B200_BLOCK_SANDWICH && s.ff_kind != B200_FF_NONE && s.ff_kind != B200_FF_DENSE_GATED) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: feed-forward kind %d", l, s.ff_kind);
         if (s.ff_kind == B200_FF_DENSE_GATED && (s.ff_dim <= 0 || (s.ff_act != B200_ACT_GELU_TANH && s.ff_act != B200_ACT_SILU && s.ff_act != B200_ACT_RELU)))
             return fail(p, B200_ERR_BAD_ARG, "layer %d: feed-forward width %d / activation %d", l, s.ff_dim, s.ff_act);
         if (s.ff_kind == B200_FF_DENSE_GATED && s.ff_dim > Y.maxF) Y.maxF = s.ff_dim;
@@ -630,18 +706,26 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         if (s.window > Y.max_window) Y.max_window = s.window;
         if (s.value_dim > Y.max_att_dv) Y.max_att_dv = s.value_dim;
     }
+    if (c.side_dim > 0) { // gate rows in whole tcgen05 tiles; their FP32 result takes the projection buffer
+        Y.side_pad = (c.side_dim + 127) / 128 * 128;
+        if (Y.side_pad > Y.maxP) Y.maxP = Y.side_pad;
+    }
     {
         int maxK = E > Y.maxO ? E : Y.maxO;
+        if (Y.maxD > maxK) maxK = Y.maxD; // reduction width of W_x
+        if (c.side_dim > maxK) maxK = c.side_dim;
         if (Y.maxF > maxK) maxK = Y.maxF;
         for (const LyLayer &L : Y.layers) if (L.s.kv_rank > maxK) maxK = L.s.kv_rank; // reduction width of the per-head value expansion
         if (Y.maxRq > maxK) maxK = Y.maxRq;
         size_t need = (size_t)maxK * 4;
-        if (outn && (size_t)2 * E * 4 > need) need = (size_t)2 * E * 4; // the row kernel holds the row and the sublayer's output
+        if ((outn || Y.maxTop > 0) && (size_t)2 * E * 4 > need) need = (size_t)2 * E * 4; // the row kernel holds the row and the sublayer's output
         for (const LyLayer &L : Y.layers) if (ly_att_smem(L.s, 0) > need) need = ly_att_smem(L.s, 0);
         if (need > (size_t)Y.smem_max) return fail(p, B200_ERR_UNSUPPORTED, "a row of %zu bytes (widest activation or window) exceeds the %d bytes of shared memory a CTA can hold", need, Y.smem_max);
         static bool attrs = false; // per function and process-wide, like plan.cu's set_smem_attrs
         if (!attrs) {
-            CK(set_max_dyn(ly::k_norm_rows, Y.smem_max));
+            CK(set_max_dyn(ly::k_norm_rows<LY_NORM_THREADS>, Y.smem_max));
+            CK(set_max_dyn(ly::k_norm_rows<1024>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<64, 32>, Y.smem_max));
             CK(set_max_dyn(ly::k_block_norm_rows<LY_NORM_THREADS>, Y.smem_max));
             CK(set_max_dyn(ly::k_block_norm_rows<1024>, Y.smem_max));
             CK(set_max_dyn(ly::k_moe_route<float>, Y.smem_max));
@@ -704,6 +788,10 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     if ((rc = dalloc(p, &Y.head, (size_t)c.vocab_size * E * 2))) return rc;
     if ((rc = ly_mat(p, tensors, nt, "head", c.vocab_size, E, Y.head, 0))) return rc;
     if (lnb && (rc = ly_layernorm_embedding(p, tensors, nt))) return rc;
+    if (c.side_dim > 0) {
+        if ((rc = dalloc(p, &Y.side_emb, (size_t)c.vocab_size * c.n_layers * c.side_dim * 2))) return rc;
+        if ((rc = ly_mat(p, tensors, nt, "side.embed", c.vocab_size, c.n_layers * c.side_dim, Y.side_emb, 0))) return rc;
+    }
     if (outn || lnb) {
         if ((rc = ly_vec_f32(p, tensors, nt, "final.norm", E, &Y.final_norm))) return rc;
     } else if (Y.prenorm) {
@@ -736,6 +824,15 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             if ((rc = ly_vec_f32(p, tensors, nt, pre + "norm1", E, &L.norm1))) return rc;
             if ((rc = ly_vec_f32(p, tensors, nt, pre + "norm1b", E, &L.norm1b))) return rc;
         }
+        if (c.side_dim > 0 && (rc = ly_side_upload(p, l, L, tensors, nt))) return rc;
+        if (s.ff_kind == B200_FF_DENSE_PLAIN || s.ff_kind == B200_FF_MOE) { // sandwich blocks only
+            if ((rc = ly_vec_f32(p, tensors, nt, pre + "norm2", E, &L.norm2))) return rc;
+            if ((rc = ly_vec_f32(p, tensors, nt, pre + "norm2b", E, &L.norm2b))) return rc;
+            if ((rc = ly_sandwich_ff_upload(p, l, L, tensors, nt))) return rc;
+        }
+        if (s.mixer == B200_MIXER_LIGHTNING || s.mixer == B200_MIXER_ATTENTION_SCAN) {
+            if ((rc = ly_sandwich_mixer_upload(p, l, L, tensors, nt))) return rc;
+        } else {
         if ((rc = dalloc(p, &L.w_proj, (size_t)L.P * E * 2))) return rc;
         if (L.P > L.Pn) CK(cudaMemset(L.w_proj + (size_t)L.Pn * E, 0, (size_t)(L.P - L.Pn) * E * 2));
         if ((rc = ly_mat(p, tensors, nt, mx + "q", L.qd, E, L.w_proj, 0))) return rc;
@@ -800,6 +897,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         } // windowed attention
         if ((rc = dalloc(p, &L.w_o, (size_t)E * L.gd * 2))) return rc;
         if ((rc = ly_mat(p, tensors, nt, mx + "o", E, L.gd, L.w_o, 0))) return rc;
+        } // windowed attention, gated delta rule
         if (s.ff_kind == B200_FF_DENSE_GATED) {
             const int F = s.ff_dim;
             if (Y.prenorm) {
@@ -855,6 +953,10 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             CK(cudaMemset(R.cstate, 0, cb));
             continue;
         }
+        if (L.s.mixer == B200_MIXER_LIGHTNING || L.s.mixer == B200_MIXER_ATTENTION_SCAN) {
+            if ((rc = ly_sandwich_run(p, R, L))) return rc;
+            if (L.s.mixer == B200_MIXER_LIGHTNING) continue;
+        }
         R.kw = L.kd; R.vw = L.vd;
         if ((rc = dalloc(p, &R.kc, (size_t)Y.ring * L.kd * 4))) return rc;
         if ((rc = dalloc(p, &R.vc, (size_t)Y.ring * L.vd * 4))) return rc;
@@ -862,7 +964,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         CK(cudaMemset(R.vc, 0, (size_t)Y.ring * L.vd * 4));
         // tensor-core prefill attention: BF16 plans, key = value size 64 or 128, a window whose tiles fit shared memory
         const int kind = ly_mma_kind(L.mixprep ? L.dk_eff : L.s.key_dim, L.s.value_dim);
-        if (!Y.f32 && Y.att_mma && Y.cap > 1 && kind && ly_mma_smem(kind, L.s.window) <= (size_t)Y.smem_max && Y.maxP % 4 == 0) {
+        if (!Y.f32 && Y.att_mma && Y.cap > 1 && kind && ly_mma_smem(kind, L.s.window) <= (size_t)Y.smem_max && Y.maxP % 4 == 0 && L.gd % 2 == 0) {
             if ((rc = dalloc(p, &R.kc16, (size_t)Y.ring * L.kd * 2))) return rc;
             if ((rc = dalloc(p, &R.vc16, (size_t)Y.ring * L.vd * 2))) return rc;
             CK(cudaMemset(R.kc16, 0, (size_t)Y.ring * L.kd * 2));
@@ -884,8 +986,19 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         if (!Y.f32 && Y.maxD > 0 && (rc = dalloc(p, &Y.U16, cap * Y.maxD * 2))) return rc;
         if (Y.maxDO > 0 && !Y.DO && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
     }
-    if (lnb && Y.maxDO > 0 && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
-    if (Y.maxD > 0 && ((rc = dalloc(p, &Y.DLT, cap * Y.maxD * 4)) || (rc = dalloc(p, &Y.DO, cap * (Y.maxDO > 0 ? Y.maxDO : 1) * 4)))) return rc;
+    if (Y.maxDO > 0 && !Y.DO && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
+    if (Y.maxD > 0 && (rc = dalloc(p, &Y.DLT, cap * Y.maxD * 4))) return rc;
+    if (Y.maxX > 0) { // attention + scan
+        if ((rc = dalloc(p, &Y.XP, cap * Y.maxX * 4))) return rc;
+        if (!Y.f32 && ((rc = dalloc(p, &Y.U16, cap * Y.maxD * 2)) || (rc = dalloc(p, &Y.DT16, cap * Y.maxRank * 2)))) return rc;
+        CK(cudaStreamCreateWithFlags(&Y.branch, cudaStreamNonBlocking));
+        CK(cudaEventCreateWithFlags(&Y.ev_fork, cudaEventDisableTiming));
+        CK(cudaEventCreateWithFlags(&Y.ev_join, cudaEventDisableTiming));
+    }
+    if (c.side_dim > 0) {
+        if ((rc = dalloc(p, &Y.SIDE32, rows32 * c.side_dim * 4))) return rc;
+        if (!Y.f32 && (rc = dalloc(p, &Y.SIDE16, cap * c.side_dim * 2))) return rc;
+    }
     if ((rc = dalloc(p, &Y.Y, cap * E * 4))) return rc;
     if ((rc = dalloc(p, &Y.PROJ, cap * Y.maxP * 4))) return rc;
     if ((rc = dalloc(p, &Y.A32, rows32 * E * 4))) return rc;
@@ -896,7 +1009,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         if ((rc = dalloc(p, &Y.ATT16, cap * Y.maxO * 2))) return rc;
         if ((rc = dalloc(p, &Y.H16, cap * slots * maxF * 2))) return rc;
     }
-    if (par || outn || lnb) {
+    if (par || outn || lnb || Y.maxTop > 0) {
         if (Y.maxKX > 0) {
             if ((rc = dalloc(p, &Y.KX16, (size_t)Y.ring * Y.maxKX * 2))) return rc;
             if ((rc = dalloc(p, &Y.VX16, (size_t)Y.ring * Y.maxVX * 2))) return rc;
@@ -1027,7 +1140,7 @@ static int ly_batch(b200_plan *p, const int32_t *tokens, int n, int start_pos, c
             ly::NormArgs a{};
             a.x = Y.X; a.w_pre = Y.final_norm; a.gather = Y.rows; a.eps = Y.c.norm_eps; a.E = E; a.w_off = Y.w_off;
             a.out32 = Y.f32 ? Y.A32 : nullptr; a.out16 = Y.f32 ? nullptr : Y.A16;
-            if ((rc = launch_k(p, false, ly::k_norm_rows, dim3(m), dim3(LY_NORM_THREADS), (size_t)E * 4, a))) return rc;
+            if ((rc = launch_k(p, false, ly::k_norm_rows<LY_NORM_THREADS>, dim3(m), dim3(LY_NORM_THREADS), (size_t)E * 4, a))) return rc;
         }
         LyTc t_head;
         if (Y.tc_head) { t_head.a = &Y.m_a; t_head.b = &Y.m_head; t_head.c = &Y.m_log_c; }

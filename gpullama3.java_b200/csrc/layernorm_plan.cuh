@@ -45,7 +45,7 @@ static int ly_layernorm_sizes(b200_plan *p, int l, LyLayer &L, const b200_layer_
             return fail(p, B200_ERR_BAD_ARG, "layer %d: feed-forward width %d / activation %d", l, s.ff_dim, s.ff_act);
     } else if (s.ff_kind == B200_FF_MOE) {
         if (s.moe_router != B200_MOE_SOFTMAX_CHOSEN || s.moe_identity || s.moe_shared_ff) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: router kind %d in this block", l, s.moe_router);
-        if (s.ff_dim <= 0 || s.ff_experts <= 0 || s.ff_top <= 0 || s.ff_top > s.ff_experts || (size_t)(E + 2 * s.ff_experts) * 4 > (size_t)Y.smem_max ||
+        if (s.ff_dim <= 0 || s.ff_experts <= 0 || s.ff_top <= 0 || s.ff_top > s.ff_experts || (size_t)(E + 3 * s.ff_experts) * 4 > (size_t)Y.smem_max ||
             (s.moe_plain ? s.ff_act != B200_ACT_RELU2 : s.ff_act != B200_ACT_SILU && s.ff_act != B200_ACT_GELU_TANH))
             return fail(p, B200_ERR_BAD_ARG, "layer %d: %d experts of width %d, %d chosen, activation %d", l, s.ff_experts, s.ff_dim, s.ff_top, s.ff_act);
         if (s.ff_top > Y.maxTop) Y.maxTop = s.ff_top;

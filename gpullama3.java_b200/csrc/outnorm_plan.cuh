@@ -100,7 +100,7 @@ static int ly_outnorm_sizes(b200_plan *p, int l, LyLayer &L, const b200_layer_sp
         const int XI = s.ff_experts + s.moe_identity;
         if (s.moe_router != B200_MOE_SOFTMAX_OUTPUT) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: router kind %d in this block", l, s.moe_router);
         if (s.ff_dim <= 0 || s.ff_experts < 0 || s.moe_identity < 0 || XI <= 0 || s.ff_top <= 0 || s.ff_top > XI || s.ff_act != B200_ACT_SILU || s.moe_shared_ff < 0 ||
-            (size_t)(E + 2 * (XI + 1)) * 4 > (size_t)Y.smem_max)
+            (size_t)(E + 3 * (XI + 1)) * 4 > (size_t)Y.smem_max)
             return fail(p, B200_ERR_BAD_ARG, "layer %d: %d experts + %d identity experts of width %d, %d chosen, activation %d", l, s.ff_experts, s.moe_identity, s.ff_dim, s.ff_top, s.ff_act);
         if (s.ff_dim > Y.maxF) Y.maxF = s.ff_dim;
         if (s.moe_shared_ff > Y.maxF) Y.maxF = s.moe_shared_ff;
@@ -399,7 +399,7 @@ static int ly_enqueue_outnorm(b200_plan *p, bool decode, int n, const StepState 
             }
             if (rc) return rc;
             if ((rc = launch_k(p, false, ly::k_gated_group_norm, dim3(n), dim3(n == 1 && inner >= 2048 ? 1024 : 256), (size_t)inner * 4, (const float *)Y.DO, Y.maxDO, (const float *)Y.PROJ, Y.maxP, (const float *)L.onorm, inner,
-                               s.mixer_norm_groups, Y.c.norm_eps, att32, att16, L.gd))) return rc;
+                               s.mixer_norm_groups, Y.c.norm_eps, 0, att32, att16, L.gd))) return rc;
             nl += 3;
         }
         if ((rc = ly_project<ly::EPI_STORE>(p, decode, n, Y.ATT32, Y.ATT16, L.w_o, nullptr, E, L.gd, Y.Y, nullptr, E, 0, &t_o))) return rc;
@@ -416,7 +416,7 @@ static int ly_enqueue_outnorm(b200_plan *p, bool decode, int n, const StepState 
                 if (Y.tc && h16 && L.tc_gu) { // tcgen05 product into the FP32 projection buffer, then the activation into the next operand
                     LyTc t_up; t_up.a = &Y.m_a; t_up.b = &L.m_up; t_up.c = &Y.m_proj_c;
                     if ((rc = ly_project<ly::EPI_STORE>(p, false, n, nullptr, Y.A16, L.w_gu, nullptr, F, E, Y.PROJ, nullptr, Y.maxP, 0, &t_up))) return rc;
-                    if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, (const float *)Y.PROJ, Y.maxP, F, s.ff_act, Y.H16, F))) return rc;
+                    if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, (const float *)Y.PROJ, Y.maxP, F, s.ff_act, Y.H16, F, ly::TokenGate{}))) return rc;
                     nl += 2;
                 } else {
                     if ((rc = ly_project<ly::EPI_ACT>(p, decode, n, x32, Y.A16, L.w_gu, nullptr, F, E, Y.H32, h16 ? Y.H16 : nullptr, F, s.ff_act))) return rc;

@@ -21,7 +21,7 @@ constexpr int BM = 128, BK = 64, BN = 128;
 // Epilogue modes: F32 store (QKV), F32 read-add-store (x += A*W^T: Wo and W2), and the gate/up pair:
 // the B tile is 64 rows of W1 and 64 rows of W3 for the same 64 hidden units, so accumulator columns
 // [0,64) = gate, [64,128) = up, and the epilogue emits f16(silu(gate)*up) (InferenceCore.java:150-158).
-// GEMM_ACT (single-CTA kernel): a plain product with an activation, bf16(act(C)).
+// GEMM_ACT (single-CTA and persistent CTA-pair kernel): a plain product with an activation, bf16(act(C)).
 enum { GEMM_F32 = 0, GEMM_RESID = 1, GEMM_GATEUP = 2, GEMM_ACT = 3 };
 
 __device__ __forceinline__ uint32_t s32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -599,6 +599,29 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(256, 1)
                                 const float g0 = __uint_as_float(g[8 * v + 2 * e]), g1 = __uint_as_float(g[8 * v + 2 * e + 1]);
                                 w[e] = gated_pair(flavor, g0, g1, __uint_as_float(u[8 * v + 2 * e]), __uint_as_float(u[8 * v + 2 * e + 1]));
                             }
+                            dst[v] = make_uint4(w[0], w[1], w[2], w[3]);
+                        }
+                    }
+                }
+            } else if (MODE == GEMM_ACT) {
+                __nv_bfloat16 *C = reinterpret_cast<__nv_bfloat16 *>(Cv);
+#pragma unroll 1
+                for (int c0 = 0; c0 < BN; c0 += 32) {
+                    uint32_t r[32];
+                    tmem_ld32(tlane + (uint32_t)c0, r);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (c0 + 32 >= BN) { // last TMEM read of this tile
+                        asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                        __syncwarp();
+                        if (lane == 0) mbar_arrive_leader(tempty0 + 8 * buf);
+                    }
+                    if (row < m_valid) {
+                        uint4 *dst = reinterpret_cast<uint4 *>(C + (size_t)row * ldc + n0 + c0);
+#pragma unroll
+                        for (int v = 0; v < 4; v++) {
+                            uint32_t w[4];
+#pragma unroll
+                            for (int e = 0; e < 4; e++) w[e] = act_pair(flavor, __uint_as_float(r[8 * v + 2 * e]), __uint_as_float(r[8 * v + 2 * e + 1]));
                             dst[v] = make_uint4(w[0], w[1], w[2], w[3]);
                         }
                     }

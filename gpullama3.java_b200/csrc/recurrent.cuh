@@ -12,7 +12,7 @@
 //                        output S * gelu_tanh(y): a two-level scan over the rows of a chunk (up to 32 row groups per CTA);
 //   * k_ssd_scan         state-space recurrence with a matrix state per head, S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x,
 //                        state columns in registers;
-//   * k_gated_group_norm y * silu(z), RMS norm in groups, weight;
+//   * k_gated_group_norm y * silu(z), RMS norm in groups, weight (or: RMS norm, weight, then * sigmoid(z));
 //   * k_slice_norm_rope  RMS norm of every key_dim slice of q and k with one weight, table-driven rotation, key / value rows into the ring;
 //   * k_diff_combine     differential attention: o = a1 - lambda a2, o / rms(o) * (1 - diff) per head;
 //   * k_act_rows         activation over FP32 rows into the operand buffer of the next GEMM.
@@ -234,10 +234,14 @@ __global__ void __launch_bounds__(256) k_shift_rows(const float *__restrict__ x,
     }
 }
 
-// Activation over FP32 rows: out[r][i] = act(in[r * ldi + i]), i < F.  grid (n), 256 threads.
-__global__ void __launch_bounds__(256) k_act_rows(const float *__restrict__ in, int ldi, int F, int act, bf16 *__restrict__ out16, int ldo) {
+// Activation over FP32 rows: out[r][i] = act(in[r * ldi + i]) (times the entry of the row's token, with a table), i < F.  grid (n), 256 threads.
+__global__ void __launch_bounds__(256) k_act_rows(const float *__restrict__ in, int ldi, int F, int act, bf16 *__restrict__ out16, int ldo, TokenGate tg) {
     const int r = blockIdx.x;
-    for (int i = threadIdx.x; i < F; i += 256) out16[(size_t)r * ldo + i] = __float2bfloat16_rn(act_apply(act, in[(size_t)r * ldi + i]));
+    for (int i = threadIdx.x; i < F; i += 256) {
+        float v = act_apply(act, in[(size_t)r * ldi + i]);
+        if (tg.table) v *= token_gate(tg, r, i);
+        out16[(size_t)r * ldo + i] = __float2bfloat16_rn(v);
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -529,23 +533,26 @@ __global__ void __launch_bounds__(SSD_THREADS) k_ssd_scan(const float *__restric
     for (int i = 0; i < R; i++) Sg[(size_t)i * SSD_THREADS] = s[i];
 }
 
-// out = GN(y * silu(z); w) with GN an RMS norm in `groups` equal consecutive parts of the row (n_in entries).  One CTA per row (any
-// multiple of 32 threads), dynamic shared memory: n_in floats.
+// out = GN(y * silu(z); w) with GN an RMS norm in `groups` equal consecutive parts of the row (n_in entries); sigmoid_after: out = GN(y; w) * sigmoid(z).
+// One CTA per row (any multiple of 32 threads), dynamic shared memory: n_in floats.
 __global__ void __launch_bounds__(1024) k_gated_group_norm(const float *__restrict__ Yv, int ldy, const float *__restrict__ Z, int ldz, const float *__restrict__ w, int n_in,
-                                                          int groups, float eps, float *__restrict__ out32, bf16 *__restrict__ out16, int ldo) {
+                                                          int groups, float eps, int sigmoid_after, float *__restrict__ out32, bf16 *__restrict__ out16, int ldo) {
     extern __shared__ __align__(16) float gv[];
     __shared__ float red[32];
     __shared__ float inv[LY_OUTNORM_MAX_GROUPS];
     const int r = blockIdx.x;
     for (int i = threadIdx.x; i < n_in; i += blockDim.x) {
+        const float y = Yv[(size_t)r * ldy + i];
+        if (sigmoid_after) { gv[i] = y; continue; }
         const float z = Z[(size_t)r * ldz + i];
-        gv[i] = Yv[(size_t)r * ldy + i] * (z / (1.0f + expf(-z)));
+        gv[i] = y * (z / (1.0f + expf(-z)));
     }
     __syncthreads();
     group_inv_rms(gv, n_in, groups, eps, inv, red);
     const int part = n_in / groups;
     for (int i = threadIdx.x; i < n_in; i += blockDim.x) {
-        const float v = gv[i] * inv[i / part] * w[i];
+        float v = gv[i] * inv[i / part] * w[i];
+        if (sigmoid_after) v *= sigmoidf_(Z[(size_t)r * ldz + i]);
         if (out32) out32[(size_t)r * ldo + i] = v;
         if (out16) out16[(size_t)r * ldo + i] = __float2bfloat16_rn(v);
     }

@@ -26,6 +26,7 @@ ARCH_LATUSUN = 4
 ARCH_LEROSUN = 5
 ARCH_DINUZEN = 6
 ARCH_KEGASUN = 7
+ARCH_ZULESUN = 8
 
 GGML_BF16 = 30  # ggml's id for bfloat16; layered plans take their safetensors tensors under it
 _SAFETENSORS_TYPES = {"BF16": GGML_BF16, "F16": GGMLType.F16, "F32": GGMLType.F32}
@@ -104,12 +105,23 @@ class LayerSpec:
     # mixture of experts
     moe_router: str = "sigmoid_input"   # | "softmax_output": softmax scores, selection by score + correction, weights on the outputs
     #                                     | "softmax_chosen": selection by logit + bias, softmax over the chosen logits on the outputs
+    #                                     | "softmax_groups": softmax scores, selection inside the best groups, scores as weights on the outputs
     moe_identity: int = 0               # identity experts behind the real ones
     moe_scale: float = 1.0
     moe_shared_ff: int = 0              # width of the shared expert (0: none)
     moe_plain: bool = False             # experts without a gate: down(act(up x))
     q_rank: int = 0                     # latent attention: > 0: queries through a normed latent of that size
     gate_cap: float = 0.0               # "mlstm": soft cap of both gates' logits
+    mask_chunked: bool = False          # attention sees its own chunk of `window` positions (counted from position 0) instead of the last `window`
+    rope_factor: float = 0.0            # > 0: rotation frequencies divided by it
+    decay: tuple = ()                   # "lightning": constant decay per head
+    # "attention_scan": an attention (the fields above) beside a selective scan over scan_inner channels of scan_state states, steps through scan_rank entries
+    scan_inner: int = 0
+    scan_state: int = 0
+    scan_rank: int = 0
+    branch_scale: tuple = (1.0, 1.0)    # factors of the attention's and the scan's result
+    moe_groups: int = 0                 # "softmax_groups": equal groups of neighbouring experts, of which the moe_keep best are eligible
+    moe_keep: int = 0
 
 
 @dataclass
@@ -136,6 +148,7 @@ class LayeredConfiguration:
     # "layernorm": x += mixer(LN x); x += ff(LN x), layer norms with a weight and no bias
     bigram: tuple | None = None  # (buckets, factor of the previous token, factor of the token): a hashed row added to the embedding
     sinusoid_base: float = 0.0   # > 0: a sinusoidal position vector added to the embedding
+    side_dim: int = 0            # > 0: per-layer token input of that many gated entries behind every layer
 
     @property
     def n_layers(self):
@@ -372,10 +385,53 @@ def kegasun_configuration(cfg: dict, tensor_shapes: dict, context_length: int) -
         block="layernorm", bigram=(int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])) if bg else None, sinusoid_base=10000.0)
 
 
+def zulesun_configuration(cfg: dict, tensor_shapes: dict, context_length: int) -> LayeredConfiguration:
+    """config.json of a Zulesun model -> LayeredConfiguration: sandwich-normed blocks; per layer a decayed linear attention or a chunk-masked
+    attention beside a selective scan, and a squared-ReLU feed-forward, a mixture of gated SiLU experts behind a group-limited softmax
+    router, or none; a per-layer token input behind every layer.  All sizes and all model-dependent constants are read from the file."""
+    layers = []
+    for i, lc in enumerate(cfg["layers"]):
+        m, mlp = lc["mixer"], lc.get("mlp")
+        if mlp is None:
+            ff = dict(ff_dim=0)
+        elif mlp.get("kind") == "dense":
+            ff = dict(ff_dim=int(mlp["ff"]), ff_act="relu2", ff_kind="dense_plain")
+        elif mlp.get("kind") == "moe":
+            r = mlp["router"]
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            ff = dict(ff_dim=int(mlp["expert"]["ff"]), ff_act="silu", ff_kind="moe", ff_experts=int(r["experts"]), ff_top=int(r["top"]),
+                      moe_router="softmax_groups", moe_groups=int(g["count"]), moe_keep=int(g["keep"]))
+        else:
+            raise UnsupportedModel(f"layer {i}: feed-forward kind {mlp.get('kind')!r}")
+        base = dict(bias_rows=0, bias_far=0.0, sink=False, gate=True, qkv_bias=False)
+        if lc["type"] == "lightning":
+            decay = tuple(float(d) for d in m["decay"])
+            if len(decay) != int(m["heads"]):
+                raise UnsupportedModel(f"layer {i}: {len(decay)} decays for {m['heads']} heads")
+            layers.append(LayerSpec(heads=int(m["heads"]), kv_heads=int(m["heads"]), key_dim=int(m["dim"]), value_dim=int(m["vdim"]), window=1, score_scale=1.0, softcap=0.0,
+                                    qk_norm=False, mixer="lightning", decay=decay, **base, **ff))
+        elif lc["type"] == "parallel":
+            a, s = m["left"], m["right"]
+            rot, mask = a.get("rot"), a.get("mask")
+            sc = (rot or {}).get("scaling")
+            layers.append(LayerSpec(
+                heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), key_dim=int(a["dim"]), value_dim=int(a["vdim"]), window=int(mask["size"]) if mask else int(context_length),
+                mask_chunked=mask is not None, score_scale=float(a["scale"]), softcap=float(a.get("softcap") or 0.0), qk_norm=True,
+                rope_dims=int(rot["dims"]) if rot else 0, rope_layout="half", rope_base=float(rot["base"]) if rot else 10000.0, rope_factor=float(sc["factor"]) if sc else 0.0,
+                mixer="attention_scan", conv_taps=int(s["conv"]), scan_inner=int(s["inner"]), scan_state=int(s["state"]), scan_rank=int(s["dt_rank"]),
+                branch_scale=(float(m["left_scale"]), float(m["right_scale"])), **base, **ff))
+        else:
+            raise UnsupportedModel(f"layer {i}: mixer type {lc['type']!r} (Zulesun layers are 'lightning' or 'parallel')")
+    side = cfg.get("token_side")
+    return LayeredConfiguration(
+        ARCH_ZULESUN, int(cfg["width"]), int(cfg["vocab"]), int(context_length), float(cfg["norm"]["eps"]), float(cfg["embedding"]["scale"]), layers, None,
+        block="sandwich", side_dim=int(side["dim"]) if side else 0)
+
+
 # config.json "architecture" -> (model type, configuration builder): the registry of safetensors model directories
 CONFIG_ARCHITECTURES = {"Pibidra": ("PIBIDRA", pibidra_configuration), "Latusun": ("LATUSUN", latusun_configuration),
                         "Lerosun": ("LEROSUN", lerosun_configuration), "Dinuzen": ("DINUZEN", dinuzen_configuration),
-                        "Kegasun": ("KEGASUN", kegasun_configuration)}
+                        "Kegasun": ("KEGASUN", kegasun_configuration), "Zulesun": ("ZULESUN", zulesun_configuration)}
 DEFAULT_LAYERED_CONTEXT = 4096
 
 

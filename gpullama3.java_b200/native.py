@@ -43,7 +43,9 @@ class LayerSpec(C.Structure):
                [(n, C.c_int32) for n in ("ff_experts", "ff_top", "value_from_key", "head_temp", "head_mix", "conv_taps", "score_maps")] + \
                [("diff_init", C.c_float)] + \
                [(n, C.c_int32) for n in ("qk_head_norm", "mixer_norm_groups", "moe_router", "moe_identity")] + \
-               [("moe_scale", C.c_float), ("moe_shared_ff", C.c_int32), ("q_rank", C.c_int32), ("gate_cap", C.c_float), ("moe_plain", C.c_int32)]
+               [("moe_scale", C.c_float), ("moe_shared_ff", C.c_int32), ("q_rank", C.c_int32), ("gate_cap", C.c_float), ("moe_plain", C.c_int32)] + \
+               [("mask_chunked", C.c_int32), ("rope_factor", C.c_float)] + [(n, C.c_int32) for n in ("scan_inner", "scan_state", "scan_rank")] + \
+               [("branch_scale", C.c_float * 2), ("moe_groups", C.c_int32), ("moe_keep", C.c_int32)]
 
 
 class LayeredConfig(C.Structure):
@@ -52,14 +54,14 @@ class LayeredConfig(C.Structure):
                [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "compute", "block")] + \
                [("residual_mult", C.c_float), ("logit_softcap", C.c_float)] + \
                [(n, C.c_int32) for n in ("norm_groups", "token_shift", "depth_average", "bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "sinusoid")] + \
-               [("sinusoid_base", C.c_float)]
+               [("sinusoid_base", C.c_float), ("side_dim", C.c_int32)]
 
 
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
 ACTIVATIONS = {"gelu_tanh": 0, "silu": 1, "relu": 2, "gelu_erf": 3, "relu2": 4}
-MIXERS = {"window_attention": 1, "latent_attention": 2, "gated_delta": 3, "rglru": 4, "ssd": 5, "mlstm": 6}
+MIXERS = {"window_attention": 1, "latent_attention": 2, "gated_delta": 3, "rglru": 4, "ssd": 5, "mlstm": 6, "lightning": 7, "attention_scan": 8}
 FF_KINDS = {"none": 0, "dense": 1, "moe": 2, "dense_plain": 3}
-MOE_ROUTERS = {"sigmoid_input": 0, "softmax_output": 1, "softmax_chosen": 2}
+MOE_ROUTERS = {"sigmoid_input": 0, "softmax_output": 1, "softmax_chosen": 2, "softmax_groups": 3}
 ROPE_LAYOUTS = {"half": 0, "interleaved": 1}
 BLOCKS = {"sandwich": 0, "parallel": 1, "prenorm": 2, "outnorm": 3, "layernorm": 4}
 

@@ -13,6 +13,7 @@ import os
 import numpy as np
 
 from . import native
+from .gguf import GGMLType
 from .loader import Model
 
 
@@ -71,6 +72,7 @@ def make_layered_config(model: Model, compute: str = "bfloat16"):
         b, mp, mc = c.bigram
         cfg.bigram_buckets, cfg.bigram_mul_prev, cfg.bigram_mul_cur = b, mp % b, mc % b
     cfg.sinusoid, cfg.sinusoid_base = int(c.sinusoid_base > 0.0), c.sinusoid_base
+    cfg.side_dim = c.side_dim
     specs = []
     for s in c.layers:
         if s.mixer not in native.MIXERS:
@@ -92,8 +94,21 @@ def make_layered_config(model: Model, compute: str = "bfloat16"):
         sp.score_maps, sp.diff_init, sp.qk_head_norm, sp.mixer_norm_groups = s.score_maps, s.diff_init, int(s.qk_head_norm), s.mixer_norm_groups
         sp.moe_router, sp.moe_identity, sp.moe_scale, sp.moe_shared_ff = native.MOE_ROUTERS[s.moe_router], s.moe_identity, s.moe_scale, s.moe_shared_ff
         sp.q_rank, sp.gate_cap, sp.moe_plain = s.q_rank, s.gate_cap, int(s.moe_plain)
+        sp.mask_chunked, sp.rope_factor = int(s.mask_chunked), s.rope_factor
+        sp.scan_inner, sp.scan_state, sp.scan_rank = s.scan_inner, s.scan_state, s.scan_rank
+        sp.branch_scale[:] = s.branch_scale
+        sp.moe_groups, sp.moe_keep = s.moe_groups, s.moe_keep
         specs.append(sp)
     return cfg, specs
+
+
+def layered_constants(model: Model) -> dict:
+    """Per-head constants of a layered configuration that reach the plan as FP32 tensors beside the model's own."""
+    out = {}
+    for i, s in enumerate(model.configuration.layers):
+        if s.decay:
+            out[f"l{i}.mix.decay"] = (GGMLType.F32, (len(s.decay),), np.asarray(s.decay, dtype="<f4").view(np.uint8))
+    return out
 
 
 def make_config(model: Model, fp16_lanes: int | None = None) -> native.Config:
@@ -122,7 +137,7 @@ class B200MasterPlan:
             if tp_size > 1:
                 raise native.UnsupportedOperation(-2, "layered plans are single-GPU")
             cfg, specs = make_layered_config(model, compute)
-            self._native = native.NativePlan(cfg, model.tensors, max(1, self.prefill_batch_size), device, layer_specs=specs)
+            self._native = native.NativePlan(cfg, model.tensors | layered_constants(model), max(1, self.prefill_batch_size), device, layer_specs=specs)
             return
         cfg = make_config(model, fp16_lanes)
         cfg.tp_rank, cfg.tp_size = tp_rank, tp_size

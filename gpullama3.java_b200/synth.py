@@ -828,3 +828,110 @@ def kegasun_model(cfg: dict, weights: dict, context_length: int):
     tensors = {k: (loader.GGML_BF16, tuple(reversed(v.shape)), bf16_bits(v).view(np.uint8).reshape(-1)) for k, v in weights.items()}
     config = loader.kegasun_configuration(cfg, {k: v.shape for k, v in weights.items()}, context_length)
     return loader.Model(None, config, "KEGASUN", tensors)
+
+
+# ---- Zulesun: sandwich-normed blocks of decayed linear attention and chunk-masked attention beside a selective scan, with a token input per layer ----
+def zulesun_lightning(heads: int, key_dim: int, value_dim: int, mlp: dict | None = None, decay: list | None = None) -> dict:
+    """A decayed-linear-attention entry of config.json's "layers" (decay = None: one factor per head, spread between fast and slow)."""
+    if decay is None:
+        decay = [float(1.0 - 0.5 ** (1.0 + 7.0 * (h + 0.5) / heads)) for h in range(heads)]
+    return {"type": "lightning", "mixer": {"heads": heads, "dim": key_dim, "vdim": value_dim, "decay": [float(d) for d in decay]}, "mlp": mlp}
+
+
+def zulesun_parallel(heads: int, kv_heads: int, key_dim: int, value_dim: int, chunk: int, inner: int, state: int, dt_rank: int, taps: int, mlp: dict | None = None, *,
+                     rot_dims: int | None = None, base: float = 10000.0, factor: float | None = 4.0, scale: float | None = None, softcap: float = 25.0,
+                     branch_scale: tuple = (0.9, 1.2)) -> dict:
+    """An attention + selective scan entry (factor = None: rotation without scaling)."""
+    rot = {"dims": key_dim // 4 * 2 if rot_dims is None else rot_dims, "base": float(base)}
+    if factor is not None:
+        rot["scaling"] = {"factor": float(factor)}
+    return {"type": "parallel",
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": key_dim, "vdim": value_dim, "mask": {"size": chunk}, "rot": rot,
+                               "scale": float(key_dim ** -0.5 if scale is None else scale), "softcap": float(softcap)},
+                      "left_scale": float(branch_scale[0]),
+                      "right": {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": taps}, "right_scale": float(branch_scale[1])},
+            "mlp": mlp}
+
+
+def zulesun_dense(ff: int) -> dict:
+    return {"kind": "dense", "ff": ff}
+
+
+def zulesun_moe(experts: int, top: int, ff: int, groups: int = 1, keep: int = 1) -> dict:
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+
+
+def zulesun_config(width: int, vocab: int, layers: list, side: int | None = 12, eps: float = 1e-5, scale: float | None = None) -> dict:
+    """side = entries of the per-layer token input (None: none)."""
+    cfg = {"architecture": "Zulesun", "width": width, "vocab": vocab, "embedding": {"scale": float(width ** 0.5 if scale is None else scale)}, "norm": {"eps": float(eps)}, "layers": layers}
+    if side is not None:
+        cfg["token_side"] = {"dim": side}
+    return cfg
+
+
+def zulesun_weights(cfg: dict, seed: int = 0) -> dict:
+    """name -> float32 array in the shapes the loader expects (linear weights [out][in]); BF16-representable values."""
+    from .safetensors import bf16_bits, bf16_to_f32
+
+    rng = np.random.default_rng(seed)
+    E, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def mat(o, i, gain=1.0):
+        return (rng.standard_normal((o, i)) * gain / np.sqrt(i)).astype(np.float32)
+
+    def vec(n, mean=0.0, std=1.0):
+        return (mean + std * rng.standard_normal(n)).astype(np.float32)
+
+    w["embed"] = (rng.standard_normal((V, E)) / cfg["embedding"]["scale"]).astype(np.float32)
+    side = cfg.get("token_side")
+    if side:
+        w["side.embed"] = rng.standard_normal((V, len(cfg["layers"]) * side["dim"])).astype(np.float32)
+    w["final.norm"] = vec(E, 0.0, 0.2)
+    w["head"] = mat(V, E)
+    for i, lc in enumerate(cfg["layers"]):
+        m, p = lc["mixer"], f"l{i}."
+        w[p + "norm1"], w[p + "norm1b"] = vec(E, 0.0, 0.2), vec(E, -0.3, 0.2)
+        if lc["type"] == "lightning":
+            H, dk, dv = m["heads"], m["dim"], m["vdim"]
+            w[p + "mix.q"], w[p + "mix.k"], w[p + "mix.v"] = mat(H * dk, E, 1.5), mat(H * dk, E, 1.5), mat(H * dv, E, 1.5)
+            w[p + "mix.g"], w[p + "mix.norm"] = mat(H * dv, E, 2.0), vec(H * dv, 1.0, 0.2)
+            w[p + "mix.o"] = mat(E, H * dv)
+        else:
+            a, s = m["left"], m["right"]
+            H, G, dk, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            q = p + "mix.left."
+            w[q + "q"], w[q + "k"], w[q + "v"], w[q + "g"] = mat(H * dk, E), mat(G * dk, E), mat(G * dv, E), mat(H * dv, E, 2.0)
+            w[q + "q.norm"], w[q + "k.norm"] = vec(H * dk, 1.5, 0.3), vec(G * dk, 1.5, 0.3)
+            w[q + "o"] = mat(E, H * dv)
+            I, N, Rk, K = s["inner"], s["state"], s["dt_rank"], s["conv"]
+            r = p + "mix.right."
+            w[r + "in"] = mat(2 * I, E, 1.5)
+            w[r + "conv"], w[r + "conv.b"] = (rng.standard_normal((I, K)) * 0.6).astype(np.float32), vec(I, 0.0, 0.2)
+            w[r + "x"], w[r + "dt"], w[r + "dt.b"] = mat(Rk + 2 * N, I, 2.0), mat(I, Rk), vec(I, -2.0, 1.0)
+            w[r + "A_log"], w[r + "D"] = (np.log(1.0 + np.arange(N)) + 0.5 * rng.standard_normal((I, N)) - 1.0).astype(np.float32), vec(I, 1.0, 0.3)
+            w[r + "o"] = mat(E, I)
+        mlp = lc.get("mlp")
+        if mlp is not None:
+            w[p + "norm2"], w[p + "norm2b"] = vec(E, 0.0, 0.2), vec(E, -0.3, 0.2)
+            if mlp["kind"] == "dense":
+                w[p + "mlp.up"], w[p + "mlp.down"] = mat(mlp["ff"], E), mat(E, mlp["ff"])
+            else:
+                X, F = mlp["router"]["experts"], mlp["expert"]["ff"]
+                w[p + "mlp.router"] = mat(X, E, 1.5)
+                for e in range(X):
+                    w[p + f"mlp.e{e}.gate"], w[p + f"mlp.e{e}.up"], w[p + f"mlp.e{e}.down"] = mat(F, E), mat(F, E), mat(E, F)
+        if side:
+            D = side["dim"]
+            w[p + "side.gate"], w[p + "side.proj"], w[p + "side.norm"] = mat(D, E), mat(E, D), vec(E, 0.5, 0.2)
+    return {k: bf16_to_f32(bf16_bits(v)).reshape(v.shape) for k, v in w.items()}
+
+
+def zulesun_model(cfg: dict, weights: dict, context_length: int):
+    """In-memory loader.Model (benchmarks and tests: synthetic weights never touch the disk)."""
+    from . import loader
+    from .safetensors import bf16_bits
+
+    tensors = {k: (loader.GGML_BF16, tuple(reversed(v.shape)), bf16_bits(v).view(np.uint8).reshape(-1)) for k, v in weights.items()}
+    config = loader.zulesun_configuration(cfg, {k: v.shape for k, v in weights.items()}, context_length)
+    return loader.Model(None, config, "ZULESUN", tensors)

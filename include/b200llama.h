@@ -68,6 +68,11 @@ extern "C" {
                              * learned sink and a gate per head, or a matrix memory with exponential gates (mLSTM); feed-forward: gated SiLU or a
                              * mixture of plain squared-ReLU experts weighted by the softmax over the chosen logits */
 
+#define B200_ARCH_ZULESUN 8 /* a layered design: sandwich-normed blocks (as PIBIDRA) whose mixer is a decayed linear attention with a matrix state per head
+                             * ("lightning"), or a chunk-masked softmax attention beside a selective scan over the same input, summed with two scales;
+                             * a plain squared-ReLU feed-forward or a mixture of gated SiLU experts behind a group-limited softmax router; behind every
+                             * layer a gated input made from the layer's own row of a second token embedding */
+
 /* GGML tensor type ids accepted for weights (tensor/GGMLType.java:5-20) */
 #define B200_GGML_F32 0
 #define B200_GGML_F16 1
@@ -155,6 +160,15 @@ int b200_plan_create(const b200_config *cfg, const b200_tensor *tensors, int32_t
                             * [value_dim], n [key_dim], m, all zero at position 0: m' = max(f + m, i), S <- exp(f + m - m') S + exp(i - m') k v^T, n
                             * likewise with k alone; o = S^T q / (max(|n . q|, exp(-m')) + 1e-6); o / rms(o) per head, times ".norm" [heads * value_dim]
                             * times sigmoid(W_g a), then W_o.  The state is FP32 and carried between calls */
+#define B200_MIXER_LIGHTNING 7 /* q = silu(W_q a), k = silu(W_k a) (heads x key_dim), v = silu(W_v a) (heads x value_dim); per head S <- c_h S + k v^T, o = S^T q with
+                                * the constant decays "<layer>.mix.decay" (F32 [heads]; S from zero at position 0); the concatenated heads are RMS-normed with
+                                * ONE statistic times ".norm" [heads * value_dim] times sigmoid(W_g a), then W_o.  S is FP32 and carried between calls */
+#define B200_MIXER_ATTENTION_SCAN 8 /* two mixers reading the same a, result branch_scale[0] * left + branch_scale[1] * right.  left ("<layer>.mix.left.*"): windowed or
+                                     * chunk-masked attention as WINDOW_ATTENTION with qk_norm and rotation together, optional gate.  right ("<layer>.mix.right.*"):
+                                     * selective scan over scan_inner channels: W_in a = [x | z]; x <- silu(conv(x) + ".conv.b") (".conv" [channels][conv_taps]);
+                                     * W_x x = [r: scan_rank | B: scan_state | C: scan_state]; dt = softplus(W_dt r + ".dt.b") per channel; per channel c and state n
+                                     * S <- exp(-exp(".A_log") dt) S + dt x B_n (from zero at position 0), y = <S, C> + ".D" x; W_o (y * silu(z)).  S (FP32) and the
+                                     * last conv_taps - 1 convolution inputs are carried between calls */
 #define B200_FF_NONE 0
 #define B200_FF_DENSE_GATED 1 /* down(act(gate x) * (up x)) */
 #define B200_FF_MOE 2         /* sum over the ff_top experts with the largest router scores of expert_e(s_e * x), expert = FF_DENSE_GATED without
@@ -165,6 +179,8 @@ int b200_plan_create(const b200_config *cfg, const b200_tensor *tensors, int32_t
                                    * weights s / (sum of the chosen s + 1e-20) * moe_scale multiply the experts' OUTPUTS; the last moe_identity router
                                    * outputs belong to identity experts, which return what they read and own no tensors */
 #define B200_MOE_SOFTMAX_CHOSEN 2 /* z + "<layer>.mlp.router.b"; the `top` largest; weights = softmax over the chosen logits, on the experts' OUTPUTS */
+#define B200_MOE_SOFTMAX_GROUPS 3 /* s = softmax(z) over all experts; the experts form moe_groups equal groups of neighbours, a group scores the largest s in it, only
+                                   * experts of the moe_keep best groups compete; the `top` largest s of them, weights s (not renormalised) on the experts' OUTPUTS */
 #define B200_ROPE_HALF 0        /* pair (i, i + rot_dims / 2) */
 #define B200_ROPE_INTERLEAVED 1 /* pair (2i, 2i + 1) */
 #define B200_BLOCK_SANDWICH 0 /* x += N(mixer(N x)); x += N(ff(N x)) with (1 + w)-weighted RMS norms (Pibidra) */
@@ -192,7 +208,7 @@ typedef struct b200_layer_spec {
     int32_t kv_heads;   /* key/value heads; query head h reads key/value head h / (heads / kv_heads) */
     int32_t key_dim;    /* per-head query/key size */
     int32_t value_dim;  /* per-head value size */
-    int32_t window;     /* position i sees j with 0 <= i - j < window */
+    int32_t window;     /* position i sees j with 0 <= i - j < window (mask_chunked: the chunk size) */
     int32_t bias_rows;  /* rows of the learned distance table [bias_rows][heads] ("<layer>.mix.rel"); 0 = no distance bias.
                            row(n) = n below bias_rows / 2, logarithmic up to bias_far, the last row beyond */
     float bias_far;
@@ -249,10 +265,18 @@ typedef struct b200_layer_spec {
     float gate_cap;
     /* B200_FF_MOE */
     int32_t moe_plain;      /* 1: experts without a gate, down(act(up x)) ("<layer>.mlp.e<k>.{up,down}") */
+    /* attention masks and rotation */
+    int32_t mask_chunked;   /* 1: position i sees j <= i with i / window == j / window (chunks counted from position 0) instead of the last `window` positions */
+    float rope_factor;      /* > 0: every rotation frequency is divided by it (linear scaling); 0: plain */
+    /* B200_MIXER_ATTENTION_SCAN */
+    int32_t scan_inner, scan_state, scan_rank;
+    float branch_scale[2];
+    /* B200_FF_MOE, B200_MOE_SOFTMAX_GROUPS */
+    int32_t moe_groups, moe_keep;
 } b200_layer_spec;
 
 typedef struct b200_layered_config {
-    int32_t arch;           /* B200_ARCH_PIBIDRA, B200_ARCH_LATUSUN, B200_ARCH_LEROSUN, B200_ARCH_DINUZEN, B200_ARCH_KEGASUN */
+    int32_t arch;           /* B200_ARCH_PIBIDRA, B200_ARCH_LATUSUN, B200_ARCH_LEROSUN, B200_ARCH_DINUZEN, B200_ARCH_KEGASUN, B200_ARCH_ZULESUN */
     int32_t width;
     int32_t vocab_size;
     int32_t n_layers;
@@ -273,6 +297,9 @@ typedef struct b200_layered_config {
     int32_t bigram_mul_prev, bigram_mul_cur;
     int32_t sinusoid;       /* B200_BLOCK_LAYERNORM, 1: the embedding adds sin(p base^(-2i / width)) to entry 2i and its cos to entry 2i + 1 */
     float sinusoid_base;
+    int32_t side_dim;       /* B200_BLOCK_SANDWICH, > 0: behind every layer x += R(P (gelu_tanh(G x) * e)), e = entries [l * side_dim, (l + 1) * side_dim) of row `token` of
+                               "side.embed" [vocab_size][n_layers * side_dim], G "<layer>.side.gate" [side_dim][width], P "<layer>.side.proj" [width][side_dim], R an RMS
+                               norm times "<layer>.side.norm" (weights used as stored) */
 } b200_layered_config;
 
 /* prefill_batch_size = the most tokens one b200_forward_batch_prefill / _batch_logits call takes (>= 1). */

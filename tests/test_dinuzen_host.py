@@ -31,7 +31,7 @@ def test_config_registry_and_abi_structs(pkg, tmp_path):
     assert (specs[0].mixer, specs[0].score_maps, specs[0].qk_head_norm, specs[0].rope_layout, specs[0].ff_kind) == (1, 2, 1, 1, 0)
     assert (specs[1].mixer, specs[1].mixer_norm_groups, specs[1].ff_kind, specs[1].ff_act) == (5, 3, 3, 3)
     assert (specs[2].moe_router, specs[2].moe_identity, specs[2].moe_shared_ff, specs[2].kv_from, specs[3].mixer) == (1, 2, 12, 0, 4)
-    assert ctypes.sizeof(pkg.native.LayerSpec) == 44 * 4 and ctypes.sizeof(pkg.native.LayeredConfig) == 22 * 4
+    assert ctypes.sizeof(pkg.native.LayerSpec) == 53 * 4 and ctypes.sizeof(pkg.native.LayeredConfig) == 23 * 4
     # in-memory model = on-disk model
     mm = S.dinuzen_model(cfg, w, 77)
     assert mm.configuration == c and all(np.array_equal(mm.tensors[k][2], m.tensors[k][2]) for k in m.tensors)

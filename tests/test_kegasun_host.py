@@ -30,7 +30,7 @@ def test_config_registry_and_abi_structs(pkg, tmp_path):
     assert (lc.arch, lc.block, lc.compute, lc.loop_times, lc.bigram_buckets, lc.bigram_mul_prev, lc.bigram_mul_cur, lc.sinusoid, lc.sinusoid_base) == (7, 4, 1, -1, 101, 7, 5, 1, 10000.0)
     assert (specs[0].mixer, specs[0].sink, specs[0].gate, specs[0].q_rank, specs[0].kv_from, specs[0].ff_kind, specs[0].ff_act) == (2, 2, 2, 24, -1, 1, 1)
     assert (specs[1].mixer, specs[1].gate_cap, specs[1].ff_kind, specs[1].ff_act, specs[1].moe_router, specs[1].moe_plain) == (6, 15.0, 2, 4, 2, 1)
-    assert ctypes.sizeof(pkg.native.LayerSpec) == 44 * 4 and ctypes.sizeof(pkg.native.LayeredConfig) == 22 * 4
+    assert ctypes.sizeof(pkg.native.LayerSpec) == 53 * 4 and ctypes.sizeof(pkg.native.LayeredConfig) == 23 * 4
     # in-memory model = on-disk model
     mm = S.kegasun_model(cfg, w, 77)
     assert mm.configuration == c and all(np.array_equal(mm.tensors[k][2], m.tensors[k][2]) for k in m.tensors)
