@@ -464,6 +464,89 @@ def compare_kegasun(pkg, lb, local: int, steps: int, warmup: int, sizes):
             "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "tensor_tflops": burst, "tensor_source": t_src}, "sizes": out}
 
 
+# ---- --compare zulesun: the sandwich-normed hybrid (chunk-masked attention beside a selective scan, decayed linear attention, group-limited
+# experts, a token input per layer) beside the two existing models it is closest to at equal size: Dinuzen (attention and a state-space
+# recurrence, softmax-routed gated SiLU experts, plain feed-forward) and Kegasun (a matrix memory of the same heads and sizes as the linear
+# attention, latent attention).  Same width, vocabulary, number of layers, key / value sizes, state entries of the recurrences and weights per
+# expert and dense feed-forward (plain ones carry two matrices, gated ones three: their widths are in the ratio 3 : 2).
+ZULESUN_SIZES = {
+    # width, attention heads, kv heads, key = value size, chunk, scan channels, states, step rank, linear heads, linear key, linear value, experts, chosen, groups, kept,
+    # expert ff, dense ff, token input, vocab
+    "small": (1024, 16, 4, 64, 256, 2048, 16, 64, 4, 128, 256, 8, 2, 2, 1, 1024, 3072, 128, 32768),
+    "1b-like": (2048, 16, 4, 128, 256, 4096, 16, 128, 8, 128, 256, 16, 4, 4, 2, 1536, 6144, 256, 32768),
+}
+
+
+def zulesun_compare_models(S, name: str):
+    """(Zulesun config, Dinuzen config, Kegasun config, accounting) of one compare size."""
+    E, H, G, d, C, I, N, Rk, LH, lk, lv, X, top, groups, keep, F, DF, D, V = ZULESUN_SIZES[name]
+    moe, dense = S.zulesun_moe(X, top, F, groups, keep), S.zulesun_dense(DF)
+
+    def par(mlp):
+        return S.zulesun_parallel(H, G, d, d, C, I, N, Rk, 4, mlp)
+
+    def lin(mlp):
+        return S.zulesun_lightning(LH, lk, lv, mlp)
+
+    cfg = S.zulesun_config(E, V, [par(moe), lin(dense), par(dense), lin(moe)], side=D)
+    SP, SN = 64, 128  # as many state entries as the linear attention
+    SH = LH * lk * lv // (SP * SN)
+    dmoe, ddense = S.dinuzen_moe(X, top, F), S.dinuzen_dense(DF)
+    dcfg = S.dinuzen_config(E, V, [S.dinuzen_attention(H // 2, 2, d, d, dmoe), S.dinuzen_mamba2(SH, SP, SN, 1, 4, ddense), S.dinuzen_attention(H // 2, 2, d, d, ddense),
+                                   S.dinuzen_mamba2(SH, SP, SN, 1, 4, dmoe)])
+    kmoe, kdense = S.kegasun_moe(X, top, F * 3 // 2), S.kegasun_dense(DF * 2 // 3)
+    Rq, R = E * 3 // 8, E // 4
+    kcfg = S.kegasun_config(E, V, [S.kegasun_attention(H, d, d, Rq, R, C, kmoe), S.kegasun_mlstm(LH, lk, lv, kdense), S.kegasun_attention(H, d, d, Rq, R, C, kdense), S.kegasun_mlstm(LH, lk, lv, kmoe)],
+                            bigram=None)
+    w_moe, w_dense, w_side = X * E + top * 3 * F * E, 2 * DF * E, 2 * D * E
+    w_par = ((H + G) * d + G * d + H * d + 2 * I) * E + (Rk + 2 * N) * I + I * Rk + (H * d + I) * E
+    w_lin = (2 * LH * lk + 2 * LH * lv) * E + LH * lv * E
+    d_ssd = (2 * SH * SP + 2 * SN + SH) * E + SH * SP * E
+    d_att = (H + 4) * d * E + 2 * d * E + H // 2 * d * E
+    k_att = (Rq + R + H) * E + H * d * (Rq + 2 * R) + H * d * E
+    k_mem = (2 * LH * lk + 2 * LH * lv + 2 * LH) * E + LH * lv * E
+    acct = {"streamed": 2 * (w_moe + w_dense + w_par + w_lin) + 4 * w_side, "att_mac_per_pair": 2 * H * d, "rec_mac_per_token": 3 * LH * lk * lv + 3 * I * N,
+            "d_streamed": 2 * (w_moe + w_dense + d_ssd + d_att), "d_att_mac_per_pair": H * 2 * d, "d_rec_mac_per_token": 3 * SH * SP * SN,
+            "k_streamed": 2 * (w_moe + w_dense + k_att + k_mem), "k_att_mac_per_pair": 2 * H * d, "k_rec_mac_per_token": 3 * LH * lk * (lv + 1), "window": C}
+    return cfg, dcfg, kcfg, acct
+
+
+def compare_zulesun(pkg, lb, local: int, steps: int, warmup: int, sizes):
+    hbm, hbm_src = peaks()
+    burst, sustained, t_src = tensor_peak()
+    S = pkg.synth
+    out = {}
+    for name in sizes:
+        E, V = ZULESUN_SIZES[name][0], ZULESUN_SIZES[name][-1]
+        depth, n_pp = 64, 512
+        ctx = max(depth + steps + warmup + 8, n_pp + 8)
+        toks = np.asarray(lb.synthetic_tokens(V, ctx), dtype=np.int32)
+        cfg, dcfg, kcfg, a = zulesun_compare_models(S, name)
+        C = a["window"]
+        chunked = sum(i % C + 1 for i in range(n_pp))       # visible pairs of a prompt: chunks, a window, all earlier positions
+        windowed = sum(min(i + 1, C) for i in range(n_pp))
+        pairs = n_pp * (n_pp + 1) // 2
+        row = {}
+        for key, c, weights, model, streamed, flops in (
+                ("zulesun_bfloat16", cfg, S.zulesun_weights, S.zulesun_model, a["streamed"], 2 * a["att_mac_per_pair"] * chunked + 2 * a["rec_mac_per_token"] * n_pp),
+                ("dinuzen_bfloat16", dcfg, S.dinuzen_weights, S.dinuzen_model, a["d_streamed"], 2 * a["d_att_mac_per_pair"] * pairs + 2 * a["d_rec_mac_per_token"] * n_pp),
+                ("kegasun_bfloat16", kcfg, S.kegasun_weights, S.kegasun_model, a["k_streamed"], 2 * a["k_att_mac_per_pair"] * windowed + 2 * a["k_rec_mac_per_token"] * n_pp)):
+            w = weights(c, 1234)
+            plan = pkg.B200MasterPlan.initialize_plan(model(c, w, ctx), prefill_batch_size=n_pp, device=local, compute="bfloat16")
+            row[key] = _layered_leg(plan, toks, depth, warmup, steps, n_pp, hbm, burst, 2 * (streamed + V * E), 2.0 * streamed * n_pp + 2.0 * flops,
+                                    ((0, "up_or_gate_up"), (1, "down"), (2, "fused_projection"), (3, "mixer_out"), (4, "classifier")))
+            plan.free()
+            del w
+        row["config"] = {"width": E, "vocab": V, "layers": 4, "order": "attention + scan with experts, linear attention with dense, attention + scan with dense, linear attention with experts",
+                         "sizes": dict(zip(("width", "attention_heads", "kv_heads", "key_value_size", "chunk", "scan_channels", "states", "step_rank", "linear_heads", "linear_key", "linear_value",
+                                            "experts", "chosen", "groups", "kept", "expert_ff", "dense_ff", "token_input", "vocab"), ZULESUN_SIZES[name])),
+                         "closest": "Dinuzen: attention, state space, attention, state space with as many state entries as the linear attention; Kegasun: latent attention, matrix memory of the same sizes",
+                         "decode": f"tg{steps} from depth {depth + warmup}", "prefill": f"pp{n_pp} in one chunk from depth 0"}
+        out[name] = row
+    return {"metric": "zulesun_vs_closest_models", "unit": "tok/s", "data": "synthetic", "dtype": "bf16 weights, f32 accumulate",
+            "peaks": {"hbm_gbs": hbm, "hbm_source": hbm_src, "tensor_tflops": burst, "tensor_source": t_src}, "sizes": out}
+
+
 class ClockSampler:
     """nvidia-smi clocks/throttle reasons sampled DURING the timed region."""
     Q = "clocks.sm,clocks.max.sm,power.draw,clocks_event_reasons.hw_slowdown,clocks_event_reasons.hw_thermal_slowdown," \
@@ -579,10 +662,10 @@ def main():
     ap.add_argument("--depth", type=int, default=-1, help="LlamaBench -d: KV positions filled before the timed steps (default: the warm-up steps)")
     ap.add_argument("--workload", default=WORKLOAD, choices=["llama-3-8b", "llama-3-70b", "llama-3.2-1b", "qwen3-4b"],
                     help="shape of the synthetic model (default: the BASELINE headline, Llama-3-8B; 70B is BASELINE config 5, meant for --gpus 2/4/8)")
-    ap.add_argument("--compare", default=None, choices=["pibidra", "latusun", "lerosun", "dinuzen", "kegasun"],
+    ap.add_argument("--compare", default=None, choices=["pibidra", "latusun", "lerosun", "dinuzen", "kegasun", "zulesun"],
                     help="instead of the headline workload: decode and prefill throughput of a layered design beside its closest existing model "
-                         "at equal sizes (pibidra: the FP16 Qwen3 plan; latusun, lerosun: the Pibidra plan; dinuzen: the Lerosun plan; kegasun: the Latusun and the Dinuzen plan), with per-kernel rooflines; one JSON line")
-    ap.add_argument("--compare-sizes", default=None, help="comma-separated size names (pibidra: 1b-like,8b-like; latusun: small,lite-like; lerosun, dinuzen, kegasun: small,1b-like)")
+                         "at equal sizes (pibidra: the FP16 Qwen3 plan; latusun, lerosun: the Pibidra plan; dinuzen: the Lerosun plan; kegasun: the Latusun and the Dinuzen plan; zulesun: the Dinuzen and the Kegasun plan), with per-kernel rooflines; one JSON line")
+    ap.add_argument("--compare-sizes", default=None, help="comma-separated size names (pibidra: 1b-like,8b-like; latusun: small,lite-like; lerosun, dinuzen, kegasun, zulesun: small,1b-like)")
     args = ap.parse_args()
     K, W = args.steps, max(args.warmup, 3)
     if args.compare:
@@ -593,7 +676,9 @@ def main():
         pkg = ge.import_package()
         sampler = ClockSampler(local)
         sampler.start()
-        if args.compare == "kegasun":
+        if args.compare == "zulesun":
+            line = compare_zulesun(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))
+        elif args.compare == "kegasun":
             line = compare_kegasun(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))
         elif args.compare == "dinuzen":
             line = compare_dinuzen(pkg, pkg.llama_bench, local, min(K, 64), W, (args.compare_sizes or "small,1b-like").split(","))

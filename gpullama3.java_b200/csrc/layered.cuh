@@ -567,31 +567,36 @@ __device__ __forceinline__ void rope_pair_index(int i, int dims, int layout, int
 
 // One CTA per row: projection biases, RMS statistics over the WHOLE q and the WHOLE k projection, q normalised in place,
 // k / v into the ring.
-__global__ void __launch_bounds__(256) k_qk_prep(float *__restrict__ P, int ldp, WindowAttn a, const float *__restrict__ bias, float *__restrict__ kc,
+// (a single row takes 1024 threads: more of its loads are in flight)
+template <int NTH>
+__global__ void __launch_bounds__(NTH) k_qk_prep(float *__restrict__ P, int ldp, WindowAttn a, const float *__restrict__ bias, float *__restrict__ kc,
                                                  float *__restrict__ vc, bf16 *__restrict__ kc16, bf16 *__restrict__ vc16, const StepState *__restrict__ st) {
-    __shared__ float red[32];
+    __shared__ float red[32], redk[32];
     const int r = blockIdx.x, tid = threadIdx.x;
     const int qd = a.heads * a.dk, kd = a.kv_heads * a.dk, vd = a.kv_heads * a.dv;
     float *q = P + (size_t)r * ldp, *k = q + qd, *v = k + kd;
     const int slot = (st->pos + r) % a.ring;
     if (bias) { // q | k | v biases of the fused projection, added where it is consumed
-        for (int i = tid; i < qd + kd + vd; i += 256) q[i] += bias[i];
+        for (int i = tid; i < qd + kd + vd; i += NTH) q[i] += bias[i];
         __syncthreads();
     }
     float qinv = 1.0f, kinv = 1.0f;
-    if (a.qnorm) {
-        float ss = 0.0f;
-        for (int i = tid; i < qd; i += 256) ss = fmaf(q[i], q[i], ss);
-        ss = block_sum(ss, red);
-        qinv = 1.0f / sqrtf(ss / (float)qd + a.eps);
+    if (a.qnorm || a.knorm) { // both sums in one reduction
+        float sq = 0.0f, sk = 0.0f;
+#pragma unroll 4
+        for (int i = tid; i < qd; i += NTH) sq = fmaf(q[i], q[i], sq);
+        for (int i = tid; i < kd; i += NTH) sk = fmaf(k[i], k[i], sk);
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if ((tid & 31) == 0) { red[tid >> 5] = sq; redk[tid >> 5] = sk; }
+        __syncthreads();
+        const int lane = tid & 31;
+        sq = warp_sum(lane < NTH / 32 ? red[lane] : 0.0f);
+        sk = warp_sum(lane < NTH / 32 ? redk[lane] : 0.0f);
+        if (a.qnorm) qinv = 1.0f / sqrtf(sq / (float)qd + a.eps);
+        if (a.knorm) kinv = 1.0f / sqrtf(sk / (float)kd + a.eps);
     }
-    if (a.knorm) {
-        float ss = 0.0f;
-        for (int i = tid; i < kd; i += 256) ss = fmaf(k[i], k[i], ss);
-        ss = block_sum(ss, red);
-        kinv = 1.0f / sqrtf(ss / (float)kd + a.eps);
-    }
-    for (int i = tid; i < vd; i += 256) {
+    for (int i = tid; i < vd; i += NTH) {
         vc[(size_t)slot * vd + i] = v[i];
         if (vc16) vc16[(size_t)slot * vd + i] = __float2bfloat16_rn(v[i]);
     }
@@ -610,7 +615,7 @@ __global__ void __launch_bounds__(256) k_qk_prep(float *__restrict__ P, int ldp,
             if (hd < a.heads) return a.qnorm ? x * qinv * a.qnorm[at] : x;
             return a.knorm ? x * kinv * a.knorm[at - qd] : x;
         };
-        for (int e = tid; e < (a.heads + a.kv_heads) * half; e += 256) {
+        for (int e = tid; e < (a.heads + a.kv_heads) * half; e += NTH) {
             const int hd = e / half, i = e % half;
             int u, w;
             rope_pair_index(i, a.rope_dims, a.rope_layout, u, w);
@@ -618,14 +623,14 @@ __global__ void __launch_bounds__(256) k_qk_prep(float *__restrict__ P, int ldp,
             emit(hd, u, fmaf(xu, co, -(xw * si)));
             emit(hd, w, fmaf(xw, co, xu * si));
         }
-        for (int e = tid; e < (a.heads + a.kv_heads) * rest; e += 256) {
+        for (int e = tid; e < (a.heads + a.kv_heads) * rest; e += NTH) {
             const int hd = e / rest, i = a.rope_dims + e % rest;
             emit(hd, i, normed(hd, i));
         }
         return;
     }
-    for (int i = tid; i < qd; i += 256) q[i] = a.qnorm ? q[i] * qinv * a.qnorm[i] : q[i];
-    for (int i = tid; i < kd; i += 256) {
+    for (int i = tid; i < qd; i += NTH) q[i] = a.qnorm ? q[i] * qinv * a.qnorm[i] : q[i];
+    for (int i = tid; i < kd; i += NTH) {
         const float kv = a.knorm ? k[i] * kinv * a.knorm[i] : k[i];
         kc[(size_t)slot * kd + i] = kv;
         if (kc16) kc16[(size_t)slot * kd + i] = __float2bfloat16_rn(kv); // BF16 twin row for the tensor-core prefill attention
@@ -819,6 +824,8 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const unsigned *>(&v);
 }
+// 1 / (1 + exp(-x)) with the hardware exponential and division: relative error ~1e-6, far below the BF16 rounding of the gated result
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
 // tanh(x) = 1 - 2 / (1 + exp(2x)) with the hardware exponential: absolute error ~1e-7, far below the BF16 rounding of the
 // operands that produced x (the FP32 kernels keep tanhf)
 __device__ __forceinline__ float tanh_fast(float x) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x)); }
@@ -1012,8 +1019,8 @@ __global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(con
             float v0 = o[j][2 * rr] * inv * ghead, v1 = o[j][2 * rr + 1] * inv * ghead;
             if (a.gate && !a.gate_heads) {
                 const float2 gv = *reinterpret_cast<const float2 *>(gate + d);
-                v0 *= 1.0f / (1.0f + expf(-gv.x));
-                v1 *= 1.0f / (1.0f + expf(-gv.y));
+                v0 *= sigmoid_fast(gv.x);
+                v1 *= sigmoid_fast(gv.y);
             }
             if (out32) *reinterpret_cast<float2 *>(out32 + (size_t)r * ldo + (size_t)h * DV + d) = make_float2(v0, v1); // FP32 results (what a later subtraction reads)
             else *reinterpret_cast<unsigned *>(out + (size_t)r * ldo + (size_t)h * DV + d) = pack_bf16(v0, v1);

@@ -88,6 +88,7 @@ struct LyLayer {
     // lightning: decays per head.  Attention + scan: ad = the attention's output columns (gd = ad + scan_inner), x_off = first scan column of a projection
     // row ([x | z]), W_x with nx rows (nxp with padding), W_dt, decay exponents; conv_w, conv_b, dt_bias, ssd_d as above
     float *decay = nullptr, *a2 = nullptr;
+    bool chunkwise = false; // lightning: BF16 prefill on the tensor cores
     int ad = 0, x_off = 0, nx = 0, nxp = 0;
     ly::bf16 *w_x = nullptr, *w_dt = nullptr;
     CUtensorMap m_wx, m_u, m_wdt, m_dt16;
@@ -171,6 +172,8 @@ struct Layered {
     float *XP = nullptr;
     ly::bf16 *DT16 = nullptr;
     int maxX = 0, maxRank = 0;
+    ly::bf16 *LQ16 = nullptr; // lightning: q | k | v of a chunk behind their activation
+    int maxLQ = 0;
     CUtensorMap m_xp_c, m_dt_c;
     cudaStream_t branch = nullptr;
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
@@ -356,7 +359,8 @@ static int ly_enqueue_attention(b200_plan *p, bool decode, int n, const StepStat
         rc = launch_k(p, false, ly::k_rope_mix_prep, dim3(n, (L.s.heads + hpc - 1) / hpc + 1), dim3(ROPE_MIX_THREADS), (size_t)(L.qd > L.kd ? L.qd : L.kd) * 4, (const float *)Y.PROJ, Y.maxP, ra,
                       (const float *)L.b_proj, Y.Q, ldq, R.kc, R.vc, R.kc16, R.vc16, st, hpc);
     } else
-        rc = launch_k(p, false, ly::k_qk_prep, dim3(n), dim3(256), (size_t)0, Y.PROJ, Y.maxP, wa, (const float *)L.b_proj, R.kc, R.vc, R.kc16, R.vc16, st);
+        rc = n == 1 && L.qd + L.kd >= 1024 ? launch_k(p, false, ly::k_qk_prep<1024>, dim3(1), dim3(1024), (size_t)0, Y.PROJ, Y.maxP, wa, (const float *)L.b_proj, R.kc, R.vc, R.kc16, R.vc16, st)
+           : launch_k(p, false, ly::k_qk_prep<256>, dim3(n), dim3(256), (size_t)0, Y.PROJ, Y.maxP, wa, (const float *)L.b_proj, R.kc, R.vc, R.kc16, R.vc16, st);
     if (rc) return rc;
     ++*nl;
     const size_t asm_ = ly_att_smem(L.s, Y.ring);
@@ -740,6 +744,11 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             CK(set_max_dyn(ly::k_window_attention_mma<128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<256, 128>, Y.smem_max));
             CK(set_max_dyn(ly::k_delta_prep, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<32, 16>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 16>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<64>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<128>, Y.smem_max));
             CK(set_max_dyn(ly::k_rope_mix_prep, Y.smem_max));
             CK(set_max_dyn(ly::k_delta_rule, Y.smem_max));
             CK(set_max_dyn(ly::k_outnorm_rows<LY_NORM_THREADS>, Y.smem_max));
@@ -988,6 +997,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     }
     if (Y.maxDO > 0 && !Y.DO && (rc = dalloc(p, &Y.DO, cap * Y.maxDO * 4))) return rc;
     if (Y.maxD > 0 && (rc = dalloc(p, &Y.DLT, cap * Y.maxD * 4))) return rc;
+    if (Y.maxLQ > 0 && (rc = dalloc(p, &Y.LQ16, cap * Y.maxLQ * 2))) return rc;
     if (Y.maxX > 0) { // attention + scan
         if ((rc = dalloc(p, &Y.XP, cap * Y.maxX * 4))) return rc;
         if (!Y.f32 && ((rc = dalloc(p, &Y.U16, cap * Y.maxD * 2)) || (rc = dalloc(p, &Y.DT16, cap * Y.maxRank * 2)))) return rc;

@@ -3,7 +3,13 @@
 // Per head, over the rows of a launch, S [dk][dv] carried from launch to launch (zero at position 0), c a constant of the head:
 //     q = silu(q'), k = silu(k'), v = silu(v');   S <- c S + k v^T;   o = S^T q
 //   * k_lightning_scan<R>  token by token in FP32, the state in registers: sixteen lanes share a column of S, lane `slice` holds R of its rows
-//                          (ssd_rows); projections staged through shared memory with the activation applied on the way.
+//                          (ssd_rows); projections staged through shared memory with the activation applied on the way;
+//   * k_lightning_chunk<DK>  the same for a prefill chunk of BF16 plans, on the tensor cores (mma.sync m16n8k16): q, k, v rounded to BF16 behind their
+//                          activation (what a BF16 plan may do), 64 tokens at a time
+//                              o_t = sum_{s <= t} c^(t-s) <q_t, k_s> v_s + c^(t+1) S^T q_t,   S <- c^64 S + sum_s c^(63-s) k_s v_s^T.
+//                          Everything behind the activations stays 32-bit: scores and decays are FP32, S accumulates in FP32 registers, and every FP32
+//                          operand of a product (decayed score, decayed value, S) enters as the sum of two BF16 numbers (its rounding and the
+//                          rounding of the rest, 16 bits together) against an exact BF16 operand.
 // The state is kept as its transpose, [head][dv][lightning_rows(dk)] floats: a column is contiguous (rows beyond dk stay zero).
 // The read-out is finished by k_gated_group_norm.
 #pragma once
@@ -130,6 +136,189 @@ __global__ void __launch_bounds__(LIGHT_THREADS) k_lightning_scan(const float *_
     } else {
 #pragma unroll
         for (int i = 0; i < R; i++) Sg[slice * R + i] = s[i];
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// grid (heads, ceil(dv / LC_COLS)), LC_THREADS threads, dynamic shared memory lightning_chunk_smem(DK).  QKV [n][ld]: [q: heads * DK | k: heads * DK |
+// v: heads * dv] behind the activation; dv a multiple of 8, ld a multiple of 8.  A CTA walks the chunk's tokens LC_TOKENS at a time (next tile in flight by
+// cp.async) for LC_COLS columns of one head's state.  Warp w: read-out of token rows 16 (w & 3) .. for 32 of the columns; state columns
+// (rows of the transpose) 16 (w & 3) .. for half of the DK entries, as accumulator fragments of the update product.
+// ---------------------------------------------------------------------------------------------------------------------
+#define LC_TOKENS 64
+#define LC_COLS 64
+#define LC_THREADS 256
+template <int DK> __host__ __device__ constexpr size_t lightning_chunk_smem() { // Q, K x 2 buffers, V x 2, split decayed V, split S^T
+    return (size_t)2 * (4 * LC_TOKENS * (DK + 8) + 2 * LC_TOKENS * (LC_COLS + 8) + 2 * LC_TOKENS * (LC_COLS + 8) + 2 * LC_COLS * (DK + 8));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void *row) {
+    const unsigned a = (unsigned)__cvta_generic_to_shared(row);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+// x, y -> packed BF16 roundings and packed roundings of what they leave
+__device__ __forceinline__ void split_bf16(float x, float y, unsigned &hi, unsigned &lo) {
+    hi = pack_bf16(x, y);
+    lo = pack_bf16(x - bf_lo(hi), y - bf_hi(hi));
+}
+
+template <int DK>
+__global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__restrict__ QKV, int ld, LightningArgs a, float *__restrict__ S, int n, const StepState *__restrict__ st,
+                                                                float *__restrict__ Y, int ldy) {
+    extern __shared__ __align__(16) unsigned char lsm[];
+    constexpr int T = LC_TOKENS, QW = DK + 8, VW = LC_COLS + 8;
+    typedef bf16 QRow[QW];
+    typedef bf16 VRow[VW];
+    QRow *Qs = reinterpret_cast<QRow *>(lsm), *Ks = Qs + 2 * T; // [buffer * T + token]
+    QRow *SH = Ks + 2 * T, *SL = SH + LC_COLS;                 // [state column]
+    VRow *Vs = reinterpret_cast<VRow *>(SL + LC_COLS), *VH = Vs + 2 * T, *VL = VH + T;
+    __shared__ float pw[T + 1]; // powers of the head's decay
+    const int h = blockIdx.x, j0 = blockIdx.y * LC_COLS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int rb = (warp & 3) * 16, half = warp >> 2;
+    const int qo = h * DK, ko = a.heads * DK + h * DK, vo = 2 * a.heads * DK + h * a.dv + j0;
+    auto fetch = [&](int t0, int buf) {
+        const int nt = n - t0 < T ? n - t0 : T;
+        for (int e = tid; e < T * (DK / 8); e += LC_THREADS) {
+            const int r = e / (DK / 8), c = (e % (DK / 8)) * 8;
+            const bool ok = r < nt;
+            const bf16 *row = QKV + (size_t)(ok ? t0 + r : 0) * ld;
+            cp_async16(&Qs[buf * T + r][c], row + qo + c, ok);
+            cp_async16(&Ks[buf * T + r][c], row + ko + c, ok);
+        }
+        for (int e = tid; e < T * (LC_COLS / 8); e += LC_THREADS) {
+            const int r = e / (LC_COLS / 8), c = (e % (LC_COLS / 8)) * 8;
+            const bool ok = r < nt && j0 + c < a.dv;
+            cp_async16(&Vs[buf * T + r][c], ok ? QKV + (size_t)(t0 + r) * ld + vo + c : QKV, ok);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(0, 0);
+    if (tid <= T) pw[tid] = powf(a.decay[h], (float)tid);
+    // S^T rows j0 + rb + g (+ 8), entries half * DK / 2 + i * 8 + 2 t (+ 1)
+    float s[DK / 16][4];
+    float *Sg = S + ((size_t)h * a.dv + j0 + rb + g) * DK + half * (DK / 2) + 2 * t;
+    const bool in0 = j0 + rb + g < a.dv, in1 = j0 + rb + g + 8 < a.dv, fresh = st->pos == 0;
+#pragma unroll
+    for (int i = 0; i < DK / 16; i++) {
+        const float2 z = make_float2(0.0f, 0.0f);
+        const float2 u = in0 && !fresh ? *reinterpret_cast<const float2 *>(Sg + i * 8) : z, v = in1 && !fresh ? *reinterpret_cast<const float2 *>(Sg + (size_t)8 * DK + i * 8) : z;
+        s[i][0] = u.x; s[i][1] = u.y; s[i][2] = v.x; s[i][3] = v.y;
+    }
+    int buf = 0;
+    for (int t0 = 0; t0 < n; t0 += T, buf ^= 1) {
+        const int nt = n - t0 < T ? n - t0 : T;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads(); // this tile has landed for every thread; the other buffer and the split operands are free
+        if (t0 + T < n) fetch(t0 + T, buf ^ 1);
+        const QRow *Q = Qs + buf * T, *K = Ks + buf * T;
+        const VRow *V = Vs + buf * T;
+#pragma unroll
+        for (int i = 0; i < DK / 16; i++) {
+            unsigned hi, lo;
+            const int c = half * (DK / 2) + i * 8 + 2 * t;
+            split_bf16(s[i][0], s[i][1], hi, lo);
+            *reinterpret_cast<unsigned *>(&SH[rb + g][c]) = hi; *reinterpret_cast<unsigned *>(&SL[rb + g][c]) = lo;
+            split_bf16(s[i][2], s[i][3], hi, lo);
+            *reinterpret_cast<unsigned *>(&SH[rb + g + 8][c]) = hi; *reinterpret_cast<unsigned *>(&SL[rb + g + 8][c]) = lo;
+        }
+        for (int e = tid; e < T * (LC_COLS / 2); e += LC_THREADS) {
+            const int r = e / (LC_COLS / 2), c = (e % (LC_COLS / 2)) * 2;
+            const unsigned v = *reinterpret_cast<const unsigned *>(&V[r][c]);
+            const float f = r < nt ? pw[nt - 1 - r] : 0.0f;
+            unsigned hi, lo;
+            split_bf16(bf_lo(v) * f, bf_hi(v) * f, hi, lo);
+            *reinterpret_cast<unsigned *>(&VH[r][c]) = hi; *reinterpret_cast<unsigned *>(&VL[r][c]) = lo;
+        }
+        __syncthreads();
+        if (rb < nt) { // read-out of this warp's sixteen tokens
+            unsigned qf[DK / 16][4];
+#pragma unroll
+            for (int kk = 0; kk < DK / 16; kk++) {
+                qf[kk][0] = *reinterpret_cast<const unsigned *>(&Q[rb + g][kk * 16 + 2 * t]);
+                qf[kk][1] = *reinterpret_cast<const unsigned *>(&Q[rb + g + 8][kk * 16 + 2 * t]);
+                qf[kk][2] = *reinterpret_cast<const unsigned *>(&Q[rb + g][kk * 16 + 2 * t + 8]);
+                qf[kk][3] = *reinterpret_cast<const unsigned *>(&Q[rb + g + 8][kk * 16 + 2 * t + 8]);
+            }
+            float o[4][4];
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+#pragma unroll
+                for (int e = 0; e < 4; e++) o[j][e] = 0.0f;
+#pragma unroll
+                for (int kk = 0; kk < DK / 16; kk++) { // what the state held before these tokens
+                    const int r = half * 32 + j * 8 + g;
+                    unsigned b[2];
+                    b[0] = *reinterpret_cast<const unsigned *>(&SH[r][kk * 16 + 2 * t]); b[1] = *reinterpret_cast<const unsigned *>(&SH[r][kk * 16 + 2 * t + 8]);
+                    mma_bf16_16816(o[j], qf[kk], b);
+                    b[0] = *reinterpret_cast<const unsigned *>(&SL[r][kk * 16 + 2 * t]); b[1] = *reinterpret_cast<const unsigned *>(&SL[r][kk * 16 + 2 * t + 8]);
+                    mma_bf16_16816(o[j], qf[kk], b);
+                }
+                const float d0 = pw[rb + g + 1], d1 = pw[rb + g + 9];
+                o[j][0] *= d0; o[j][1] *= d0; o[j][2] *= d1; o[j][3] *= d1;
+            }
+#pragma unroll
+            for (int kb = 0; kb < T / 16; kb++) { // sixteen keys at a time: scores, decay and mask, values
+                if (kb * 16 > rb) break;          // later than every token of this warp
+                float p[2][4];
+#pragma unroll
+                for (int u = 0; u < 2; u++) {
+#pragma unroll
+                    for (int e = 0; e < 4; e++) p[u][e] = 0.0f;
+#pragma unroll
+                    for (int kk = 0; kk < DK / 16; kk++) {
+                        const int r = kb * 16 + u * 8 + g;
+                        unsigned b[2];
+                        b[0] = *reinterpret_cast<const unsigned *>(&K[r][kk * 16 + 2 * t]); b[1] = *reinterpret_cast<const unsigned *>(&K[r][kk * 16 + 2 * t + 8]);
+                        mma_bf16_16816(p[u], qf[kk], b);
+                    }
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int back = rb + g + (e >> 1) * 8 - (kb * 16 + u * 8 + 2 * t + (e & 1));
+                        p[u][e] = back >= 0 ? p[u][e] * pw[back] : 0.0f;
+                    }
+                }
+                unsigned ph[4], pl[4];
+                split_bf16(p[0][0], p[0][1], ph[0], pl[0]); split_bf16(p[0][2], p[0][3], ph[1], pl[1]);
+                split_bf16(p[1][0], p[1][1], ph[2], pl[2]); split_bf16(p[1][2], p[1][3], ph[3], pl[3]);
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    unsigned b[2];
+                    ldmatrix_x2_trans(b, &V[kb * 16 + (lane & 15)][half * 32 + j * 8]);
+                    mma_bf16_16816(o[j], ph, b);
+                    mma_bf16_16816(o[j], pl, b);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const int c = j0 + half * 32 + j * 8 + 2 * t; // dv is a multiple of 8: both entries or none
+                if (c >= a.dv) continue;
+                float *y = Y + (size_t)(t0 + rb + g) * ldy + (size_t)h * a.dv + c;
+                if (rb + g < nt) *reinterpret_cast<float2 *>(y) = make_float2(o[j][0], o[j][1]);
+                if (rb + g + 8 < nt) *reinterpret_cast<float2 *>(y + (size_t)8 * ldy) = make_float2(o[j][2], o[j][3]);
+            }
+        }
+        // state: decayed, plus the products of this tile's keys and decayed values
+        const float dn = pw[nt];
+#pragma unroll
+        for (int i = 0; i < DK / 16; i++) { s[i][0] *= dn; s[i][1] *= dn; s[i][2] *= dn; s[i][3] *= dn; }
+#pragma unroll
+        for (int kk = 0; kk < T / 16; kk++) {
+            unsigned vh[4], vl[4];
+            const int r = kk * 16 + (lane >> 4) * 8 + (lane & 7), c = rb + ((lane >> 3) & 1) * 8; // four 8 x 8 blocks, transposed: [value][token]
+            ldmatrix_x4_trans(vh, &VH[r][c]);
+            ldmatrix_x4_trans(vl, &VL[r][c]);
+#pragma unroll
+            for (int i = 0; i < DK / 16; i++) {
+                unsigned b[2];
+                ldmatrix_x2_trans(b, &K[kk * 16 + (lane & 15)][half * (DK / 2) + i * 8]);
+                mma_bf16_16816(s[i], vh, b);
+                mma_bf16_16816(s[i], vl, b);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DK / 16; i++) {
+        if (in0) *reinterpret_cast<float2 *>(Sg + i * 8) = make_float2(s[i][0], s[i][1]);
+        if (in1) *reinterpret_cast<float2 *>(Sg + (size_t)8 * DK + i * 8) = make_float2(s[i][2], s[i][3]);
     }
 }
 

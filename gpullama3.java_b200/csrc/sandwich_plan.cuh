@@ -1,7 +1,8 @@
 // sandwich_plan.cuh -- host side of what sandwich-normed layers (B200_BLOCK_SANDWICH, layered_plan.cuh) offer beside windowed attention and a
 // gated feed-forward (included by layered_plan.cuh): two further mixers, two further feed-forwards and the per-layer token input.
 //
-//   lightning:       fused q | k | v | g projection -> decayed linear attention (k_lightning_scan) -> one norm over all heads, sigmoid gate -> output projection
+//   lightning:       fused q | k | v | g projection -> decayed linear attention (k_lightning_scan; chunks of BF16 plans: k_lightning_chunk) -> one norm over
+//                     all heads, sigmoid gate -> output projection
 //   attention + scan: ONE fused projection q | k | v | g | x | z of both branches; then, on two streams,
 //                       whole-projection q/k norm + rotation + ring write -> chunk-masked attention (+ gate, * branch_scale[0])
 //                       convolution + SiLU -> W_x -> [W_dt] -> selective scan (+ gate silu(z), * branch_scale[1])
@@ -54,6 +55,8 @@ static int ly_sandwich_mixer_sizes(b200_plan *p, int l, LyLayer &L) {
         L.Pn = 2 * L.qd + 2 * L.vd;
         if ((size_t)L.gd * 4 > (size_t)Y.smem_max) return fail(p, B200_ERR_UNSUPPORTED, "layer %d: a read-out row of %d values exceeds the shared memory of a CTA", l, L.gd);
         if (L.gd > Y.maxDO) Y.maxDO = L.gd;
+        L.chunkwise = !Y.f32 && Y.cap > 1 && (s.key_dim == 32 || s.key_dim == 64 || s.key_dim == 128) && s.value_dim % 8 == 0;
+        if (L.chunkwise && 2 * L.qd + L.vd > Y.maxLQ) Y.maxLQ = 2 * L.qd + L.vd;
     } else { // B200_MIXER_ATTENTION_SCAN
         if (s.sink || s.gate > 1 || s.qkv_bias || s.bias_rows || s.value_from_key || s.head_temp || s.head_mix)
             return fail(p, B200_ERR_UNSUPPORTED, "layer %d: sinks, per-head gates, biases, distance tables, key-values, head temperature and head mixing are not combined with a scan", l);
@@ -212,6 +215,7 @@ static void ly_sandwich_tc_init(b200_plan *p) {
     }
 }
 
+#define LC_CHUNK_MIN 16 // rows from which a chunk takes the tensor-core form
 // Decayed linear attention of one layer, from the projection rows in PROJ to the gated read-outs in ATT32 / ATT16.
 static int ly_enqueue_lightning(b200_plan *p, bool decode, int n, const StepState *st, const LyRun &R, const LyLayer &L, int *nl) {
     Layered &Y = *p->ly;
@@ -222,7 +226,16 @@ static int ly_enqueue_lightning(b200_plan *p, bool decode, int n, const StepStat
     a.heads = s.heads; a.dk = s.key_dim; a.dv = s.value_dim; a.q_off = 0; a.k_off = L.qd; a.v_off = 2 * L.qd; a.decay = L.decay;
     const dim3 grid(s.heads, (s.value_dim + LIGHT_COLS - 1) / LIGHT_COLS), block(LIGHT_THREADS);
     const float *P = Y.PROJ;
-    switch (ly::lightning_reg_rows(s.key_dim)) {
+    if (h16 && L.chunkwise && n >= LC_CHUNK_MIN) {
+        const int w = 2 * L.qd + L.vd;
+        if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, P, Y.maxP, w, (int)ly::ACT_SILU, Y.LQ16, w, ly::TokenGate{}))) return rc;
+        const dim3 cgrid(s.heads, (s.value_dim + LC_COLS - 1) / LC_COLS);
+        const ly::bf16 *qkv = Y.LQ16;
+        if (s.key_dim == 32) rc = launch_k(p, false, ly::k_lightning_chunk<32>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<32>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
+        else if (s.key_dim == 64) rc = launch_k(p, false, ly::k_lightning_chunk<64>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<64>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
+        else rc = launch_k(p, false, ly::k_lightning_chunk<128>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<128>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
+        ++*nl;
+    } else switch (ly::lightning_reg_rows(s.key_dim)) {
     case 1: rc = launch_k(p, false, ly::k_lightning_scan<1>, grid, block, (size_t)0, P, Y.maxP, a, R.S, n, st, Y.DO, Y.maxDO); break;
     case 2: rc = launch_k(p, false, ly::k_lightning_scan<2>, grid, block, (size_t)0, P, Y.maxP, a, R.S, n, st, Y.DO, Y.maxDO); break;
     case 4: rc = launch_k(p, false, ly::k_lightning_scan<4>, grid, block, (size_t)0, P, Y.maxP, a, R.S, n, st, Y.DO, Y.maxDO); break;
@@ -283,14 +296,17 @@ static int ly_enqueue_selective(b200_plan *p, bool decode, int n, const StepStat
     const float *U = Y.DLT, *PX = Y.XP, *DT = Y.Q, *Z = Y.PROJ + z_off;
     float *o32 = h16 ? nullptr : Y.ATT32 + L.ad;
     ly::bf16 *o16 = h16 ? Y.ATT16 + L.ad : nullptr;
-    if (lpc > 4) return launch_k(p, false, ly::k_selective_scan<32, 16>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    switch (ly::sel_reg_rows(N)) {
-    case 1: return launch_k(p, false, ly::k_selective_scan<4, 1>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    case 2: return launch_k(p, false, ly::k_selective_scan<4, 2>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    case 4: return launch_k(p, false, ly::k_selective_scan<4, 4>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    case 8: return launch_k(p, false, ly::k_selective_scan<4, 8>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    case 16: return launch_k(p, false, ly::k_selective_scan<4, 16>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    default: return launch_k(p, false, ly::k_selective_scan<4, 32>, grid, block, (size_t)0, U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    const int rr = ly::sel_reg_rows(N);
+    if (lpc > SEL_LANES) {
+        if (rr == 8) return launch_k(p, false, ly::k_selective_scan<32, 8>, grid, block, ly::sel_smem(32, 8), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+        return launch_k(p, false, ly::k_selective_scan<32, 16>, grid, block, ly::sel_smem(32, 16), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    }
+    switch (rr) {
+    case 1: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 1>, grid, block, ly::sel_smem(SEL_LANES, 1), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    case 2: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 2>, grid, block, ly::sel_smem(SEL_LANES, 2), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    case 4: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 4>, grid, block, ly::sel_smem(SEL_LANES, 4), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    case 8: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 8>, grid, block, ly::sel_smem(SEL_LANES, 8), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    default: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 16>, grid, block, ly::sel_smem(SEL_LANES, 16), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
     }
 }
 

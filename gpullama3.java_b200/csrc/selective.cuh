@@ -6,9 +6,10 @@
 //     y[c] = sum_n S[c][n] C[n] + D[c] u[c],   out[c] = out_scale * y[c] * silu(z[c])
 //   * k_selective_scan<LPC, R>  LPC lanes share a channel, each keeps R of its states in registers; the rows of a launch run in sequence,
 //                               channels in parallel over lanes and CTAs.  u, dt', z of the CTA's channels and B, C are staged TB tokens at a time
-//                               with cp.async, double buffered; four tokens are worked on together (their step sizes come from one lane each,
-//                               their read-out sums are reduced with three shuffles).  A single-row launch computes dt' itself from its factor
-//                               r and W_dt: the decode step has no launch of its own for that product.
+//                               with cp.async, double buffered; what needs no state (step size, step * u, gate) is worked out once per token and channel
+//                               in a pass over the staged batch, so that the chain from token to token is one multiply-add.  Eight tokens'
+//                               read-out sums are reduced together with seven shuffles.  A single-row launch computes dt' itself from its
+//                               factor r and W_dt: the decode step has no launch of its own for that product.
 // Everything is FP32 in both compute modes.
 #pragma once
 #include "delta.cuh"
@@ -25,11 +26,19 @@ struct SelScanArgs {
     int vec;               // 1: all row strides, column offsets, rank and N are multiples of 4 floats
 };
 #define SEL_THREADS 256
-__host__ __device__ constexpr int sel_tb(int lpc, int r) { return lpc >= 32 ? 4 : r >= 16 ? 8 : 16; } // tokens per staged batch
-// States per lane when LPC = 4 lanes share a channel (LPC = 32: 16), 0: more states than the kernel holds
-__host__ __device__ inline int sel_reg_rows(int N) { return N <= 4 ? 1 : N <= 8 ? 2 : N <= 16 ? 4 : N <= 32 ? 8 : N <= 64 ? 16 : N <= 128 ? 32 : N <= 512 ? 16 : 0; }
-__host__ __device__ inline int sel_lanes(int N) { return N <= 128 ? 4 : 32; }
+#define SEL_LANES 8
+__host__ __device__ constexpr int sel_tb(int lpc, int) { return lpc >= 32 ? 8 : 16; } // tokens per staged batch
+// States per lane when SEL_LANES lanes share a channel (up to 128 states), or a whole warp does; 0: more states than the kernel holds
+__host__ __device__ inline int sel_reg_rows(int N) { return N <= 8 ? 1 : N <= 16 ? 2 : N <= 32 ? 4 : N <= 64 ? 8 : N <= 128 ? 16 : N <= 256 ? 8 : N <= 512 ? 16 : 0; }
+__host__ __device__ inline int sel_lanes(int N) { return N <= 128 ? SEL_LANES : 32; }
 __host__ __device__ inline size_t sel_state_floats(int C, int N) { return (size_t)C * sel_lanes(N) * sel_reg_rows(N); }
+__host__ __device__ constexpr size_t sel_smem(int lpc, int r) { return (size_t)4 * sel_tb(lpc, r) * lpc * r * 4; }
+// 2^x in one instruction (relative error 2^-22; results below the normal range are zero)
+__device__ __forceinline__ float exp2_approx(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 // R consecutive floats at p (16-byte aligned when R is a multiple of 4)
 template <int R> __device__ __forceinline__ void load_run(const float *p, float (&v)[R]) {
@@ -42,14 +51,18 @@ template <int R> __device__ __forceinline__ void load_run(const float *p, float 
     }
 }
 
-// grid (ceil(C / (SEL_THREADS / LPC))).  U [n][ldu] convolved channels, PX [n][ldx] parameter rows [r | B | C], DT [n][lddt], Z [n][ldz].
+// grid (ceil(C / (SEL_THREADS / LPC))), dynamic shared memory sel_smem(LPC, R).  U [n][ldu] convolved channels, PX [n][ldx] parameter rows [r | B | C], DT [n][lddt], Z [n][ldz].
 // State: [channel][LPC * R] (states beyond N stay zero).  out32 / out16: row stride ldo, first column of this mixer.
 template <int LPC, int R>
 __global__ void __launch_bounds__(SEL_THREADS) k_selective_scan(const float *__restrict__ U, int ldu, const float *__restrict__ PX, int ldx, const float *__restrict__ DT, int lddt,
                                                                 const float *__restrict__ Z, int ldz, SelScanArgs a, float *__restrict__ S, int n, const StepState *__restrict__ st,
                                                                 float *__restrict__ out32, bf16 *__restrict__ out16, int ldo) {
     constexpr int CH = SEL_THREADS / LPC, RW = LPC * R, TB = sel_tb(LPC, R);
-    __shared__ __align__(16) float us[2][TB][CH], ds[2][TB][CH], zs[2][TB][CH], Bs[2][TB][RW], Cs[2][TB][RW];
+    __shared__ __align__(16) float us[2][TB][CH], ds[2][TB][CH], zs[2][TB][CH];
+    typedef float Row[RW];
+    extern __shared__ __align__(16) unsigned char selm[];
+    Row *const Bs = reinterpret_cast<Row *>(selm), *const Cs = Bs + 2 * TB; // [buffer * TB + token]
+    __shared__ float du[TB][CH], bs[CH], Dsm[CH];
     const int tid = threadIdx.x, l = tid % LPC, cl = tid / LPC, c0 = blockIdx.x * CH, c = c0 + cl;
     const bool live = c < a.C;
     const bool own_dt = a.w_dt != nullptr;
@@ -68,8 +81,8 @@ __global__ void __launch_bounds__(SEL_THREADS) k_selective_scan(const float *__r
                 const int t = e / (RW / 4), i = (e % (RW / 4)) * 4;
                 const bool ok = t < nt && i < a.N;
                 const float *p = PX + (size_t)(ok ? t0 + t : 0) * ldx + a.rank;
-                cp_async16(&Bs[buf][t][i], ok ? p + i : PX, ok);
-                cp_async16(&Cs[buf][t][i], ok ? p + a.N + i : PX, ok);
+                cp_async16(&Bs[buf * TB + t][i], ok ? p + i : PX, ok);
+                cp_async16(&Cs[buf * TB + t][i], ok ? p + a.N + i : PX, ok);
             }
         } else {
             for (int e = tid; e < TB * CH; e += SEL_THREADS) {
@@ -84,8 +97,8 @@ __global__ void __launch_bounds__(SEL_THREADS) k_selective_scan(const float *__r
                 const int t = e / RW, i = e % RW;
                 const bool ok = t < nt && i < a.N;
                 const float *p = PX + (size_t)(ok ? t0 + t : 0) * ldx + a.rank;
-                cp_async4(&Bs[buf][t][i], ok ? p + i : PX, ok);
-                cp_async4(&Cs[buf][t][i], ok ? p + a.N + i : PX, ok);
+                cp_async4(&Bs[buf * TB + t][i], ok ? p + i : PX, ok);
+                cp_async4(&Cs[buf * TB + t][i], ok ? p + a.N + i : PX, ok);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -101,7 +114,7 @@ __global__ void __launch_bounds__(SEL_THREADS) k_selective_scan(const float *__r
     }
 #pragma unroll
     for (int i = 0; i < R; i++) A[i] = live && l * R + i < a.N ? a.a2[(size_t)c * a.N + l * R + i] : 0.0f;
-    const float bias = live ? a.dt_bias[c] : 0.0f, Dc = live ? a.D[c] : 0.0f;
+    if (tid < CH) { bs[tid] = c0 + tid < a.C ? a.dt_bias[c0 + tid] : 0.0f; Dsm[tid] = c0 + tid < a.C ? a.D[c0 + tid] : 0.0f; }
     if (own_dt) { // dt' of the only row: a warp per channel, W_dt streamed
         const int lane = tid & 31, warp = tid >> 5;
         const bool vec = (a.rank & 7) == 0 && (((size_t)a.w_dt) & 15) == 0 && (((size_t)PX) & 15) == 0;
@@ -113,43 +126,53 @@ __global__ void __launch_bounds__(SEL_THREADS) k_selective_scan(const float *__r
         }
     }
     int buf = 0;
+    const int q = l & 7;
     for (int t0 = 0; t0 < n; t0 += TB, buf ^= 1) {
         const int nt = n - t0 < TB ? n - t0 : TB;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads(); // this batch has landed for every thread, and the other buffer's batch is consumed
         if (t0 + TB < n) fetch(t0 + TB, buf ^ 1);
-        const int q = l & 3;
-        for (int tb = 0; tb < nt; tb += 4) {
-            // lane q of every four: step size of token tb + q; a token behind the last leaves the state as it is (step 0)
-            const bool in = tb + q < nt;
-            const float u_q = us[buf][tb + q][cl];
-            const float dt_q = in ? softplusf_(ds[buf][tb + q][cl] + bias) : 0.0f, dx_q = dt_q * u_q;
-            float acc[4];
+        // per token and channel: step size, step * u, D * u, gate; a token behind the last gets step 0 and leaves the state as it is
 #pragma unroll
-            for (int k = 0; k < 4; k++) {
-                const float dt = __shfl_sync(0xffffffffu, dt_q, k, 4), dx = __shfl_sync(0xffffffffu, dx_q, k, 4);
+        for (int e = tid; e < TB * CH; e += SEL_THREADS) {
+            const int t = e / CH, i = e % CH;
+            const float u = us[buf][t][i], z = zs[buf][t][i];
+            const float dt = t < nt ? softplusf_(ds[buf][t][i] + bs[i]) : 0.0f;
+            ds[buf][t][i] = dt;
+            us[buf][t][i] = dt * u;
+            du[t][i] = Dsm[i] * u;
+            zs[buf][t][i] = z / (1.0f + expf(-z)) * a.out_scale;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int tb = 0; tb < TB; tb += 8) {
+            if (tb >= nt) break;
+            float acc[8];
+#pragma unroll
+            for (int k = 0; k < 8; k++) {
+                const float dt = ds[buf][tb + k][cl], dx = us[buf][tb + k][cl];
                 float bv[R], cv[R];
-                load_run<R>(&Bs[buf][tb + k][l * R], bv);
-                load_run<R>(&Cs[buf][tb + k][l * R], cv);
+                load_run<R>(&Bs[buf * TB + tb + k][l * R], bv);
+                load_run<R>(&Cs[buf * TB + tb + k][l * R], cv);
                 float ac = 0.0f;
 #pragma unroll
                 for (int i = 0; i < R; i++) {
-                    s[i] = fmaf(exp2f(dt * A[i]), s[i], dx * bv[i]);
+                    s[i] = fmaf(exp2_approx(dt * A[i]), s[i], dx * bv[i]);
                     ac = fmaf(s[i], cv[i], ac);
                 }
                 acc[k] = ac;
             }
-            const bool hi2 = q & 2, hi1 = q & 1;
-            float p0 = hi2 ? acc[2] : acc[0], p1 = hi2 ? acc[3] : acc[1];
-            p0 += __shfl_xor_sync(0xffffffffu, hi2 ? acc[0] : acc[2], 2);
-            p1 += __shfl_xor_sync(0xffffffffu, hi2 ? acc[1] : acc[3], 2);
-            float v = hi1 ? p1 : p0;
-            v += __shfl_xor_sync(0xffffffffu, hi1 ? p0 : p1, 1);
+            const bool h4 = q & 4, h2 = q & 2, h1 = q & 1; // lane q of every eight ends up with the sum of token tb + q
+            float p4[4], p2[2];
 #pragma unroll
-            for (int o = 4; o < LPC; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-            if (in && live && l < 4) { // lane q holds the sum of token tb + q
-                const float z = zs[buf][tb + q][cl];
-                const float o = fmaf(Dc, u_q, v) * (z / (1.0f + expf(-z))) * a.out_scale;
+            for (int k = 0; k < 4; k++) p4[k] = (h4 ? acc[k + 4] : acc[k]) + __shfl_xor_sync(0xffffffffu, h4 ? acc[k] : acc[k + 4], 4);
+#pragma unroll
+            for (int k = 0; k < 2; k++) p2[k] = (h2 ? p4[k + 2] : p4[k]) + __shfl_xor_sync(0xffffffffu, h2 ? p4[k] : p4[k + 2], 2);
+            float v = (h1 ? p2[1] : p2[0]) + __shfl_xor_sync(0xffffffffu, h1 ? p2[0] : p2[1], 1);
+#pragma unroll
+            for (int o = 8; o < LPC; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+            if (tb + q < nt && live && l < 8) {
+                const float o = (v + du[tb + q][cl]) * zs[buf][tb + q][cl];
                 const size_t at = (size_t)(t0 + tb + q) * ldo + c;
                 if (out32) out32[at] = o;
                 if (out16) out16[at] = __float2bfloat16_rn(o);

@@ -908,7 +908,7 @@ def zulesun_weights(cfg: dict, seed: int = 0) -> dict:
             r = p + "mix.right."
             w[r + "in"] = mat(2 * I, E, 1.5)
             w[r + "conv"], w[r + "conv.b"] = (rng.standard_normal((I, K)) * 0.6).astype(np.float32), vec(I, 0.0, 0.2)
-            w[r + "x"], w[r + "dt"], w[r + "dt.b"] = mat(Rk + 2 * N, I, 2.0), mat(I, Rk), vec(I, -2.0, 1.0)
+            w[r + "x"], w[r + "dt"], w[r + "dt.b"] = mat(Rk + 2 * N, I, 1.5), mat(I, Rk, 0.7), vec(I, -2.0, 1.0)
             w[r + "A_log"], w[r + "D"] = (np.log(1.0 + np.arange(N)) + 0.5 * rng.standard_normal((I, N)) - 1.0).astype(np.float32), vec(I, 1.0, 0.3)
             w[r + "o"] = mat(E, I)
         mlp = lc.get("mlp")

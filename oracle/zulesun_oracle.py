@@ -61,6 +61,12 @@ def read_safetensors(path: str) -> dict:
     return out
 
 
+# ---- products ----------------------------------------------------------------------------------------------------------
+def linear(x, w):
+    """Every product with a weight matrix [out][in] goes through here."""
+    return x @ w.T
+
+
 # ---- elementwise -------------------------------------------------------------------------------------------------------
 def sigmoid(z):
     return 1.0 / (1.0 + np.exp(-z))
@@ -108,11 +114,11 @@ def lightning_scan(q, k, v, decay):
 def mixer_lightning(h, w: dict, pre: str, m: dict, eps: float):
     T = h.shape[0]
     H, d, dv = int(m["heads"]), int(m["dim"]), int(m["vdim"])
-    q = silu(h @ w[pre + "q"].T).reshape(T, H, d)
-    k = silu(h @ w[pre + "k"].T).reshape(T, H, d)
-    v = silu(h @ w[pre + "v"].T).reshape(T, H, dv)
+    q = silu(linear(h, w[pre + "q"])).reshape(T, H, d)
+    k = silu(linear(h, w[pre + "k"])).reshape(T, H, d)
+    v = silu(linear(h, w[pre + "v"])).reshape(T, H, dv)
     o = lightning_scan(q, k, v, m["decay"]).reshape(T, H * dv)
-    return (rms_norm(o, w[pre + "norm"], eps) * sigmoid(h @ w[pre + "g"].T)) @ w[pre + "o"].T
+    return linear(rms_norm(o, w[pre + "norm"], eps) * sigmoid(linear(h, w[pre + "g"])), w[pre + "o"])
 
 
 # ---- chunked attention -------------------------------------------------------------------------------------------------
@@ -142,16 +148,16 @@ def masked_softmax(e, mask):
 def chunked_attention(h, w: dict, pre: str, m: dict, eps: float):
     T = h.shape[0]
     H, G, d, dv = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
-    q = rotate_half(rms_norm(h @ w[pre + "q"].T, w[pre + "q.norm"], eps).reshape(T, H, d), m["rot"])
-    k = rotate_half(rms_norm(h @ w[pre + "k"].T, w[pre + "k.norm"], eps).reshape(T, G, d), m["rot"])
-    v = (h @ w[pre + "v"].T).reshape(T, G, dv)
+    q = rotate_half(rms_norm(linear(h, w[pre + "q"]), w[pre + "q.norm"], eps).reshape(T, H, d), m["rot"])
+    k = rotate_half(rms_norm(linear(h, w[pre + "k"]), w[pre + "k.norm"], eps).reshape(T, G, d), m["rot"])
+    v = linear(h, w[pre + "v"]).reshape(T, G, dv)
     mask = chunk_mask(T, int(m["mask"]["size"]))
     o = np.zeros((T, H, dv))
     for a in range(H):
         g = a // (H // G)
         e = soft_cap((q[:, a] @ k[:, g].T) * float(m["scale"]), m.get("softcap"))
         o[:, a] = masked_softmax(e, mask) @ v[:, g]
-    return (o.reshape(T, H * dv) * sigmoid(h @ w[pre + "g"].T)) @ w[pre + "o"].T
+    return linear(o.reshape(T, H * dv) * sigmoid(linear(h, w[pre + "g"])), w[pre + "o"])
 
 
 # ---- selective scan ----------------------------------------------------------------------------------------------------
@@ -174,13 +180,13 @@ def selective_scan(x, dt, B, C, A, D):
 
 def mamba(h, w: dict, pre: str, m: dict):
     inner, N, rank = int(m["inner"]), int(m["state"]), int(m["dt_rank"])
-    xz = h @ w[pre + "in"].T
+    xz = linear(h, w[pre + "in"])
     x, z = xz[:, :inner], xz[:, inner:]
     x = silu(causal_conv(x, w[pre + "conv"], w[pre + "conv.b"]))
-    p = x @ w[pre + "x"].T
-    dt = softplus(p[:, :rank] @ w[pre + "dt"].T + w[pre + "dt.b"])
+    p = linear(x, w[pre + "x"])
+    dt = softplus(linear(p[:, :rank], w[pre + "dt"]) + w[pre + "dt.b"])
     y = selective_scan(x, dt, p[:, rank:rank + N], p[:, rank + N:], -np.exp(w[pre + "A_log"]), w[pre + "D"])
-    return (y * silu(z)) @ w[pre + "o"].T
+    return linear(y * silu(z), w[pre + "o"])
 
 
 def mixer_parallel(h, w: dict, pre: str, m: dict, eps: float):
@@ -189,17 +195,17 @@ def mixer_parallel(h, w: dict, pre: str, m: dict, eps: float):
 
 # ---- feed-forward ------------------------------------------------------------------------------------------------------
 def ff_dense(h, w: dict, pre: str):
-    return np.maximum(h @ w[pre + "up"].T, 0.0) ** 2 @ w[pre + "down"].T
+    return linear(np.maximum(linear(h, w[pre + "up"]), 0.0) ** 2, w[pre + "down"])
 
 
 def expert(h, w: dict, pre: str):
-    return (silu(h @ w[pre + "gate"].T) * (h @ w[pre + "up"].T)) @ w[pre + "down"].T
+    return linear(silu(linear(h, w[pre + "gate"])) * linear(h, w[pre + "up"]), w[pre + "down"])
 
 
 def moe_route(h, w: dict, pre: str, router: dict, margins=None):
     """(ids [T, top], weights [T, top]); margins (a list) receives, per token, the smaller of the two gaps that decide, in logits: between
     the worst kept and the best dropped group, and between the last chosen and the first rejected expert of the kept groups."""
-    z = h @ w[pre + "router"].T
+    z = linear(h, w[pre + "router"])
     s = np.exp(z - z.max(-1, keepdims=True))
     s /= s.sum(-1, keepdims=True)
     T, X = s.shape
@@ -237,7 +243,7 @@ def ff_moe(h, w: dict, pre: str, mlp: dict, margins=None):
 # ---- per-layer token input ---------------------------------------------------------------------------------------------
 def token_side(x, tokens, w: dict, pre: str, layer: int, dim: int, eps: float):
     e = w["side.embed"][np.asarray(tokens)][:, layer * dim:(layer + 1) * dim]
-    y = (gelu_tanh(x @ w[pre + "side.gate"].T) * e) @ w[pre + "side.proj"].T
+    y = linear(gelu_tanh(linear(x, w[pre + "side.gate"])) * e, w[pre + "side.proj"])
     return rms_norm(y, w[pre + "side.norm"], eps)
 
 
@@ -262,7 +268,7 @@ def forward(cfg: dict, w: dict, tokens, return_layers: bool = False, margins=Non
         if cfg.get("token_side"):
             x = x + token_side(x, tokens, w, pre, i, int(cfg["token_side"]["dim"]), eps)
         trace.append(x.copy())
-    logits = block_norm(x, w["final.norm"], eps) @ w["head"].T
+    logits = linear(block_norm(x, w["final.norm"], eps), w["head"])
     return (logits, np.stack(trace)) if return_layers else logits
 
 

@@ -78,18 +78,25 @@ def min_margin(O, cfg, w, toks):
     return min(m) if m else np.inf
 
 
-def rounding_shift(O, cfg, w, toks):
-    """How far rounding the norms' outputs to BF16 (what the matrix products read in BF16 mode) alone moves a logits row of the float64
-    oracle.  The lightning read-out is divided by its own size, so a row whose <k, q> nearly vanishes (above all a first token) may turn by
-    any amount under rounding; such rows compare nothing."""
-    exact = O.block_norm
+def rounding_shift(O, cfg, w, toks, bits: int = 9):
+    """How far disturbing what the weight matrices read by up to 2^-bits alone moves a logits row of the float64 oracle: three random disturbances
+    and, for the 9 bits of BF16, the rounding itself.  Read-outs that are divided by their own size turn by any amount where <k, q> or a scan's
+    result nearly vanishes (above all at first tokens); such rows compare nothing."""
+    exact = O.linear
     ref = O.forward(cfg, w, toks)
+    rng = np.random.default_rng(0)
+    worst = 0.0
     try:
-        O.block_norm = lambda v, weight, eps: bf16_values({"v": exact(v, weight, eps)})["v"].astype(np.float64)
-        got = O.forward(cfg, w, toks)
+        for k in range(0 if bits == 9 else 1, 4):
+            if k == 0:
+                O.linear = lambda x, m: exact(bf16_values({"x": x})["x"].astype(np.float64), m)
+            else:
+                O.linear = lambda x, m: exact(x * (1.0 + 2.0 ** -bits * rng.uniform(-1.0, 1.0, x.shape)), m)
+            got = O.forward(cfg, w, toks)
+            worst = max(worst, max(rel_rms(got[t], ref[t]) for t in range(len(toks))))
     finally:
-        O.block_norm = exact
-    return max(rel_rms(got[t], ref[t]) for t in range(len(toks)))
+        O.linear = exact
+    return worst
 
 
 def settled_weights(S, O, cfg, seed, toks, shift):
