@@ -200,6 +200,8 @@ static int ly_project_view(b200_plan *p, bool decode, int n, const float *a32, c
     Layered &Y = *p->ly;
     if (decode) {
         const int warps = LY_MV_THREADS / 32;
+        if (EPI != ly::EPI_GATED && yb == 1 && !mv.group && !mv.mul && !mv.in_scale && ly_few_rows(p, N, K))
+            return launch_k(p, false, ly::k_matvec_row_bf16<EPI == ly::EPI_GATED ? ly::EPI_STORE : EPI>, dim3(N), dim3(LY_MV_THREADS), (size_t)0, W, a32, c32, K, act, mv.tg);
         return launch_k(p, false, ly::k_matvec_bf16<EPI>, dim3((N + warps - 1) / warps, yb), dim3(LY_MV_THREADS), (size_t)K * 4, W, (const float *)nullptr, a32, c32, N, K, act, mv);
     }
     dim3 grid((N + 63) / 64, tiles > 0 ? tiles : (n + 63) / 64, zb);

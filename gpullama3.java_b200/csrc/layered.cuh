@@ -32,6 +32,11 @@ enum { ACT_GELU_TANH = 0, ACT_SILU = 1, ACT_RELU = 2, ACT_GELU_ERF = 3, ACT_RELU
 __device__ __forceinline__ float bf_lo(unsigned v) { return __uint_as_float(v << 16); }
 __device__ __forceinline__ float bf_hi(unsigned v) { return __uint_as_float(v & 0xffff0000u); }
 
+__device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const unsigned *>(&v);
+}
+
 __device__ __forceinline__ float act_apply(int act, float z) {
     if (act == ACT_SILU) return z / (1.0f + expf(-z));
     if (act == ACT_NONE) return z;
@@ -213,21 +218,123 @@ __global__ void __launch_bounds__(NTH) k_norm_rows(NormArgs a) {
 // ---------------------------------------------------------------------------------------------------------------------
 #define LY_MV_THREADS 256
 
+// acc + eight consecutive products of a row's packed BF16 entries and x (16-byte aligned), in order
+__device__ __forceinline__ float dot8_bf16(const int4 &q, const float *x, float acc) {
+    const float4 x0 = *reinterpret_cast<const float4 *>(x), x1 = *reinterpret_cast<const float4 *>(x + 4);
+    acc = fmaf(bf_lo((unsigned)q.x), x0.x, acc); acc = fmaf(bf_hi((unsigned)q.x), x0.y, acc);
+    acc = fmaf(bf_lo((unsigned)q.y), x0.z, acc); acc = fmaf(bf_hi((unsigned)q.y), x0.w, acc);
+    acc = fmaf(bf_lo((unsigned)q.z), x1.x, acc); acc = fmaf(bf_hi((unsigned)q.z), x1.y, acc);
+    acc = fmaf(bf_lo((unsigned)q.w), x1.z, acc); acc = fmaf(bf_hi((unsigned)q.w), x1.w, acc);
+    return acc;
+}
 __device__ __forceinline__ float dot_row_bf16(const bf16 *__restrict__ w, const float *xs, int K, int lane, bool vec) {
     float acc = 0.0f;
     if (vec) {
-        for (int k = lane * 8; k < K; k += 256) {
-            const int4 q = ldg128_stream(w + k);
-            const float4 x0 = *reinterpret_cast<const float4 *>(xs + k), x1 = *reinterpret_cast<const float4 *>(xs + k + 4);
-            acc = fmaf(bf_lo((unsigned)q.x), x0.x, acc); acc = fmaf(bf_hi((unsigned)q.x), x0.y, acc);
-            acc = fmaf(bf_lo((unsigned)q.y), x0.z, acc); acc = fmaf(bf_hi((unsigned)q.y), x0.w, acc);
-            acc = fmaf(bf_lo((unsigned)q.z), x1.x, acc); acc = fmaf(bf_hi((unsigned)q.z), x1.y, acc);
-            acc = fmaf(bf_lo((unsigned)q.w), x1.z, acc); acc = fmaf(bf_hi((unsigned)q.w), x1.w, acc);
+        int k = lane * 8;
+        for (; k + 768 < K; k += 1024) { // four 128-bit loads of the row in flight per lane
+            int4 q[4];
+#pragma unroll
+            for (int u = 0; u < 4; u++) q[u] = ldg128_stream(w + k + 256 * u);
+#pragma unroll
+            for (int u = 0; u < 4; u++) acc = dot8_bf16(q[u], xs + k + 256 * u, acc);
         }
+        for (; k < K; k += 256) acc = dot8_bf16(ldg128_stream(w + k), xs + k, acc);
     } else {
         for (int k = lane; k < K; k += 32) acc = fmaf(__bfloat162float(w[k]), xs[k], acc);
     }
     return warp_sum(acc);
+}
+
+// The same for rows of whole float4 without a pass prologue or an embedding norm: every thread keeps VPT float4 of the row in registers, and the loads of the
+// row, of the sublayer output and of both weights are in flight together (the statistics are the only places where the CTA waits).
+// E a multiple of 4, at most 4 * NTH * VPT; top <= LY_NORM_TERMS.  No dynamic shared memory.
+template <int NTH, int VPT>
+__global__ void __launch_bounds__(NTH) k_norm_rows_reg(NormArgs a) {
+    __shared__ float red[32];
+    __shared__ size_t s_row[LY_NORM_TERMS];
+    __shared__ float s_wt[LY_NORM_TERMS];
+    const int r = blockIdx.x, tid = threadIdx.x, E = a.E;
+    const size_t src = (size_t)(a.gather ? a.gather[r] : r) * E, dst = (size_t)r * E;
+    if (a.ys) {
+        if (tid < a.top) {
+            const size_t e = (size_t)r * a.top + tid;
+            s_row[tid] = (a.ys_map ? (size_t)a.ys_map[e] : e) * E;
+            s_wt[tid] = a.wts[e];
+        }
+        __syncthreads();
+    }
+    const bf16 *emb = a.emb ? a.emb + (size_t)(a.tokens ? a.tokens[r] : a.st->token) * E : nullptr;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 x[VPT], y[VPT], w1[VPT], w2[VPT];
+    const bool add = a.y || a.ys;
+#pragma unroll
+    for (int v = 0; v < VPT; v++) {
+        const int i = (tid + v * NTH) * 4;
+        const bool in = i < E;
+        x[v] = y[v] = w1[v] = w2[v] = zero;
+        if (!in) continue;
+        if (emb) {
+            const uint2 q = *reinterpret_cast<const uint2 *>(emb + i);
+            x[v] = make_float4(bf_lo(q.x) * a.emb_scale, bf_hi(q.x) * a.emb_scale, bf_lo(q.y) * a.emb_scale, bf_hi(q.y) * a.emb_scale);
+        } else x[v] = *reinterpret_cast<const float4 *>(a.x + src + i);
+        if (a.y) y[v] = *reinterpret_cast<const float4 *>(a.y + src + i);
+        if (add) w1[v] = *reinterpret_cast<const float4 *>(a.w_post + i);
+        if (a.w_pre) w2[v] = *reinterpret_cast<const float4 *>(a.w_pre + i);
+    }
+    if (a.ys) {
+        for (int k0 = 0; k0 < a.top; k0 += 4) { // the loads of four entries are issued before the first is used
+#pragma unroll
+            for (int v = 0; v < VPT; v++) {
+                const int i = (tid + v * NTH) * 4;
+                float4 q[4];
+#pragma unroll
+                for (int u = 0; u < 4; u++) q[u] = i < E && k0 + u < a.top ? __ldg(reinterpret_cast<const float4 *>(a.ys + s_row[k0 + u] + i)) : zero;
+#pragma unroll
+                for (int u = 0; u < 4; u++)
+                    if (k0 + u < a.top) {
+                        const float wt = s_wt[k0 + u];
+                        y[v].x = fmaf(wt, q[u].x, y[v].x); y[v].y = fmaf(wt, q[u].y, y[v].y); y[v].z = fmaf(wt, q[u].z, y[v].z); y[v].w = fmaf(wt, q[u].w, y[v].w);
+                    }
+            }
+        }
+    }
+    auto square = [](const float4 &q, float s) { return fmaf(q.x, q.x, fmaf(q.y, q.y, fmaf(q.z, q.z, fmaf(q.w, q.w, s)))); };
+    if (add) {
+        float inv = 1.0f, off = 0.0f;
+        if (!a.post_plain) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int v = 0; v < VPT; v++) ss = square(y[v], ss);
+            ss = block_sum(ss, red);
+            inv = 1.0f / sqrtf(ss / (float)E + a.eps);
+            off = a.post_off;
+        }
+#pragma unroll
+        for (int v = 0; v < VPT; v++) {
+            x[v].x += y[v].x * inv * (off + w1[v].x); x[v].y += y[v].y * inv * (off + w1[v].y);
+            x[v].z += y[v].z * inv * (off + w1[v].z); x[v].w += y[v].w * inv * (off + w1[v].w);
+        }
+    }
+    float inv = 1.0f;
+    if (a.w_pre) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int v = 0; v < VPT; v++) ss = square(x[v], ss);
+        ss = block_sum(ss, red);
+        inv = 1.0f / sqrtf(ss / (float)E + a.eps);
+    }
+#pragma unroll
+    for (int v = 0; v < VPT; v++) {
+        const int i = (tid + v * NTH) * 4;
+        if (i >= E) continue;
+        if (a.trace) *reinterpret_cast<float4 *>(a.trace + src + i) = x[v];
+        if (!a.gather && (emb || add)) *reinterpret_cast<float4 *>(a.x + src + i) = x[v];
+        if (!a.out32 && !a.out16) continue;
+        float4 o = x[v];
+        if (a.w_pre) o = make_float4(o.x * inv * (a.w_off + w2[v].x), o.y * inv * (a.w_off + w2[v].y), o.z * inv * (a.w_off + w2[v].z), o.w * inv * (a.w_off + w2[v].w));
+        if (a.out32) *reinterpret_cast<float4 *>(a.out32 + dst + i) = o;
+        if (a.out16) *reinterpret_cast<uint2 *>(a.out16 + dst + i) = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
+    }
 }
 
 // A row of a second token embedding as a factor: entry n of a result row is multiplied by table[token * ld + n].
@@ -284,6 +391,33 @@ __global__ void __launch_bounds__(LY_MV_THREADS) k_matvec_bf16(const bf16 *__res
         }
         if (lane == 0) y[n] = v;
     }
+}
+
+// The same for matrices of FEW rows (a router, the step / state parameters of a scan, a narrow gate): a CTA per row, so that the reduction width is
+// spread over all its warps instead of one.  grid (N), LY_MV_THREADS threads; plain and EPI_ACT results.
+template <int EPI>
+__global__ void __launch_bounds__(LY_MV_THREADS) k_matvec_row_bf16(const bf16 *__restrict__ W, const float *__restrict__ x, float *__restrict__ y, int K, int act, TokenGate tg) {
+    __shared__ float red[32];
+    const int n = blockIdx.x;
+    const bf16 *w = W + (size_t)n * K;
+    float acc = 0.0f;
+    if ((K & 7) == 0 && (((size_t)W) & 15) == 0 && (((size_t)x) & 15) == 0) {
+        int k = threadIdx.x * 8;
+        for (; k + LY_MV_THREADS * 8 < K; k += 2 * LY_MV_THREADS * 8) {
+            const int4 q0 = ldg128_stream(w + k), q1 = ldg128_stream(w + k + LY_MV_THREADS * 8);
+            acc = dot8_bf16(q0, x + k, acc);
+            acc = dot8_bf16(q1, x + k + LY_MV_THREADS * 8, acc);
+        }
+        if (k < K) acc = dot8_bf16(ldg128_stream(w + k), x + k, acc);
+    } else
+        for (int k = threadIdx.x; k < K; k += LY_MV_THREADS) acc = fmaf(__bfloat162float(w[k]), x[k], acc);
+    acc = block_sum(acc, red);
+    if (threadIdx.x) return;
+    if (EPI == EPI_ACT) {
+        acc = act_apply(act, acc);
+        if (tg.table) acc *= token_gate(tg, 0, n);
+    }
+    y[n] = acc;
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -815,14 +949,9 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
 // mask and the ONLINE softmax stay in FP32 registers.  The sink is the initial state of the running softmax: maximum 0,
 // denominator exp(0) = 1, no value.  Dynamic shared memory: att_mma_smem_bytes<DK, DV>(window).
 // ---------------------------------------------------------------------------------------------------------------------
-#define LY_ATT_MMA_ROWS 128 // query rows per CTA: eight warps of 16 rows share every key tile
-#define LY_ATT_MMA_THREADS (LY_ATT_MMA_ROWS * 2)
-template <int DK, int DV> __host__ __device__ constexpr size_t att_mma_smem_bytes(int window) {
+#define LY_ATT_MMA_ROWS 128 // query rows per CTA: eight warps of 16 rows share every key tile (launches of few CTAs: 64 rows, four warps, so that more SMs work)
+template <int DK, int DV> __host__ __device__ constexpr size_t att_mma_smem_bytes(int window) { // for the taller tile; the other one needs less
     return (size_t)(LY_ATT_MMA_ROWS * (DK + 8) * 2) + (size_t)(64 * (DK + 8) * 2) * 2 + (size_t)(64 * (DV + 8) * 2) * 2 + (size_t)window * 4;
-}
-__device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const unsigned *>(&v);
 }
 // 1 / (1 + exp(-x)) with the hardware exponential and division: relative error ~1e-6, far below the BF16 rounding of the gated result
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
@@ -839,12 +968,12 @@ __device__ __forceinline__ void ldmatrix_x2_trans(unsigned (&r)[2], const void *
     asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
 }
 
-template <int DK, int DV>
-__global__ void __launch_bounds__(LY_ATT_MMA_THREADS) k_window_attention_mma(const float *__restrict__ P, int ldp, WindowAttn a, const bf16 *__restrict__ kc16,
+template <int DK, int DV, int BM = LY_ATT_MMA_ROWS>
+__global__ void __launch_bounds__(BM * 2) k_window_attention_mma(const float *__restrict__ P, int ldp, WindowAttn a, const bf16 *__restrict__ kc16,
                                                                              const bf16 *__restrict__ vc16, const StepState *__restrict__ st, int n,
                                                                              bf16 *__restrict__ out, int ldo, float *__restrict__ out32 = nullptr) {
     extern __shared__ __align__(16) unsigned char smraw[];
-    constexpr int BM = LY_ATT_MMA_ROWS;
+    constexpr int LY_ATT_MMA_THREADS = BM * 2;
     constexpr int QT = BM * (DK + 8) * 2, KT = 64 * (DK + 8) * 2, VT = 64 * (DV + 8) * 2; // bytes of the Q tile, one K tile, one V tile
     bf16(*Qs)[DK + 8] = reinterpret_cast<bf16(*)[DK + 8]>(smraw);
     float *sbias = reinterpret_cast<float *>(smraw + QT + 2 * KT + 2 * VT);

@@ -273,14 +273,22 @@ static size_t ly_mma_smem(int kind, int window) {
 }
 static int ly_launch_mma(b200_plan *p, int kind, int n, int heads, int window, const float *P, int ldp, const ly::WindowAttn &wa, const ly::bf16 *k16, const ly::bf16 *v16,
                          const StepState *st, ly::bf16 *out, int ldo, float *out32 = nullptr) {
-    const dim3 grid((n + LY_ATT_MMA_ROWS - 1) / LY_ATT_MMA_ROWS, heads), block(LY_ATT_MMA_THREADS);
     const size_t sm = ly_mma_smem(kind, window);
-    if (kind == 1) return launch_k(p, false, ly::k_window_attention_mma<64, 64>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
-    if (kind == 2) return launch_k(p, false, ly::k_window_attention_mma<128, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
-    if (kind == 4) return launch_k(p, false, ly::k_window_attention_mma<128, 64>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
-    if (kind == 5) return launch_k(p, false, ly::k_window_attention_mma<256, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
-    if (kind == 6) return launch_k(p, false, ly::k_window_attention_mma<64, 32>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
-    return launch_k(p, false, ly::k_window_attention_mma<192, 128>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
+    // few tall tiles leave SMs idle: half as many rows per CTA then
+    const bool tall = (n + LY_ATT_MMA_ROWS - 1) / LY_ATT_MMA_ROWS * heads >= p->n_sms;
+    const int rows = tall ? LY_ATT_MMA_ROWS : 64;
+    const dim3 grid((n + rows - 1) / rows, heads), block(rows * 2);
+#define LY_MMA_CASE(K, DK, DV) \
+    if (kind == K) return tall ? launch_k(p, false, ly::k_window_attention_mma<DK, DV>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32) \
+                               : launch_k(p, false, ly::k_window_attention_mma<DK, DV, 64>, grid, block, sm, P, ldp, wa, k16, v16, st, n, out, ldo, out32);
+    LY_MMA_CASE(1, 64, 64)
+    LY_MMA_CASE(2, 128, 128)
+    LY_MMA_CASE(3, 192, 128)
+    LY_MMA_CASE(4, 128, 64)
+    LY_MMA_CASE(5, 256, 128)
+    LY_MMA_CASE(6, 64, 32)
+#undef LY_MMA_CASE
+    return fail(p, B200_ERR_STATE, "no tensor-core attention of kind %d", kind);
 }
 
 static ly::WindowAttn ly_attn_args(const Layered &Y, const LyLayer &L) {
@@ -301,6 +309,9 @@ static ly::WindowAttn ly_attn_args(const Layered &Y, const LyLayer &L) {
     return a;
 }
 
+// A decode projection with a warp per row would occupy less than half of the SMs and every warp walk a long row: a CTA per row then.
+static bool ly_few_rows(const b200_plan *p, int N, int K) { return (N + LY_MV_THREADS / 32 - 1) / (LY_MV_THREADS / 32) * 2 < p->n_sms && K >= 1024; }
+
 // C[n][N] = A[n][K] W^T with the epilogue EPI; decode (n == 1 through the graph) streams the rows, prefill takes a GEMM:
 // the persistent CTA-pair tcgen05 kernel (256-wide tiles) or the single-CTA one (128-wide) of prefill_gemm.cuh when the
 // shape fits and the plan computes in BF16, else the any-shape kernels of layered.cuh.
@@ -311,6 +322,8 @@ static int ly_project(b200_plan *p, bool decode, int n, const float *a32, const 
     if (decode) {
         const int warps = LY_MV_THREADS / 32;
         int grid = (N + warps - 1) / warps;
+        if (EPI != ly::EPI_GATED && !bias && ly_few_rows(p, N, K))
+            return launch_k(p, false, ly::k_matvec_row_bf16<EPI == ly::EPI_GATED ? ly::EPI_STORE : EPI>, dim3(N), dim3(LY_MV_THREADS), (size_t)0, W, a32, c32, K, act, ly::TokenGate{});
         return launch_k(p, false, ly::k_matvec_bf16<EPI>, dim3(grid), dim3(LY_MV_THREADS), (size_t)K * 4, W, bias, a32, c32, N, K, act, ly::MvView{});
     }
     if (tc && tc->a && !Y.f32) {
@@ -385,6 +398,24 @@ static int ly_enqueue_attention(b200_plan *p, bool decode, int n, const StepStat
 #include "layernorm_plan.cuh"
 #include "sandwich_plan.cuh"
 
+// The row kernel of sandwich and pre-norm blocks: rows in registers where their shape and the step allow it, else through shared memory; a single wide row
+// takes more threads.
+static int ly_launch_norm(b200_plan *p, int n, const ly::NormArgs &a) {
+    const int E = a.E;
+    if (E % 4 == 0 && E <= 4096 && !a.w_emb && !a.x0 && !a.add_x0 && !a.step && a.top <= LY_NORM_TERMS) {
+        if (n == 1 && E > 1024) {
+            if (E <= 2048) return launch_k(p, false, ly::k_norm_rows_reg<512, 1>, dim3(1), dim3(512), (size_t)0, a);
+            return launch_k(p, false, ly::k_norm_rows_reg<1024, 1>, dim3(1), dim3(1024), (size_t)0, a);
+        }
+        if (E <= 1024) return launch_k(p, false, ly::k_norm_rows_reg<LY_NORM_THREADS, 1>, dim3(n), dim3(LY_NORM_THREADS), (size_t)0, a);
+        if (E <= 2048) return launch_k(p, false, ly::k_norm_rows_reg<LY_NORM_THREADS, 2>, dim3(n), dim3(LY_NORM_THREADS), (size_t)0, a);
+        return launch_k(p, false, ly::k_norm_rows_reg<LY_NORM_THREADS, 4>, dim3(n), dim3(LY_NORM_THREADS), (size_t)0, a);
+    }
+    const size_t sm = (size_t)(a.ys ? 2 : 1) * E * 4;
+    if (n == 1 && E >= 2048) return launch_k(p, false, ly::k_norm_rows<1024>, dim3(1), dim3(1024), sm, a);
+    return launch_k(p, false, ly::k_norm_rows<LY_NORM_THREADS>, dim3(n), dim3(LY_NORM_THREADS), sm, a);
+}
+
 // Enqueue the forward of n rows on p->stream.  decode: the single-token step (row 0, position and token from *st).
 // with_head (decode only): final norm + classifier into p->logits.  Prefill leaves the finished residual rows in X.
 static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, const int *tokens, bool with_head, float *trace, int *launches) {
@@ -410,11 +441,9 @@ static int ly_enqueue(b200_plan *p, bool decode, int n, const StepState *st, con
         a.add_x0 = add_x0 ? 1 : 0; a.step = step; a.w_pre = w_pre;
         a.out32 = w_pre && !h16 ? Y.A32 : nullptr; a.out16 = (w_pre || raw) && h16 ? Y.A16 : nullptr;
         a.gather = nullptr; a.trace = pend_trace; a.eps = Y.c.norm_eps; a.E = E;
-        const size_t sm = (size_t)(pend_ys ? 2 : 1) * E * 4;
         pend_y = pend_w = pend_ys = nullptr; pend_map = nullptr; pend_top = 0; pend_off = Y.w_off; pend_trace = nullptr;
         nl++;
-        if (n == 1 && E >= 2048) return launch_k(p, false, ly::k_norm_rows<1024>, dim3(1), dim3(1024), sm, a);
-        return launch_k(p, false, ly::k_norm_rows<LY_NORM_THREADS>, dim3(n), dim3(LY_NORM_THREADS), sm, a);
+        return ly_launch_norm(p, n, a);
     };
     for (size_t r = 0; r < Y.runs.size(); r++) {
         const LyRun &R = Y.runs[r];
@@ -730,6 +759,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             CK(set_max_dyn(ly::k_norm_rows<LY_NORM_THREADS>, Y.smem_max));
             CK(set_max_dyn(ly::k_norm_rows<1024>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<64, 32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<64, 32, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_block_norm_rows<LY_NORM_THREADS>, Y.smem_max));
             CK(set_max_dyn(ly::k_block_norm_rows<1024>, Y.smem_max));
             CK(set_max_dyn(ly::k_moe_route<float>, Y.smem_max));
@@ -739,16 +769,24 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             CK(set_max_dyn(ly::k_window_attention<float>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention<ly::bf16>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<64, 64>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<64, 64, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<128, 128>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<128, 128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<192, 128>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<192, 128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<128, 64>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<128, 64, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<256, 128>, Y.smem_max));
+            CK(set_max_dyn(ly::k_window_attention_mma<256, 128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_delta_prep, Y.smem_max));
             CK(set_max_dyn(ly::k_selective_scan<32, 16>, Y.smem_max));
             CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 16>, Y.smem_max));
-            CK(set_max_dyn(ly::k_lightning_chunk<32>, Y.smem_max));
-            CK(set_max_dyn(ly::k_lightning_chunk<64>, Y.smem_max));
-            CK(set_max_dyn(ly::k_lightning_chunk<128>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<32, 32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<32, 64>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<64, 32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<64, 64>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<128, 32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_lightning_chunk<128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_rope_mix_prep, Y.smem_max));
             CK(set_max_dyn(ly::k_delta_rule, Y.smem_max));
             CK(set_max_dyn(ly::k_outnorm_rows<LY_NORM_THREADS>, Y.smem_max));
@@ -1150,7 +1188,7 @@ static int ly_batch(b200_plan *p, const int32_t *tokens, int n, int start_pos, c
             ly::NormArgs a{};
             a.x = Y.X; a.w_pre = Y.final_norm; a.gather = Y.rows; a.eps = Y.c.norm_eps; a.E = E; a.w_off = Y.w_off;
             a.out32 = Y.f32 ? Y.A32 : nullptr; a.out16 = Y.f32 ? nullptr : Y.A16;
-            if ((rc = launch_k(p, false, ly::k_norm_rows<LY_NORM_THREADS>, dim3(m), dim3(LY_NORM_THREADS), (size_t)E * 4, a))) return rc;
+            if ((rc = ly_launch_norm(p, m, a))) return rc;
         }
         LyTc t_head;
         if (Y.tc_head) { t_head.a = &Y.m_a; t_head.b = &Y.m_head; t_head.c = &Y.m_log_c; }

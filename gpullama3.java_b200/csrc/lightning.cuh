@@ -140,16 +140,14 @@ __global__ void __launch_bounds__(LIGHT_THREADS) k_lightning_scan(const float *_
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
-// grid (heads, ceil(dv / LC_COLS)), LC_THREADS threads, dynamic shared memory lightning_chunk_smem(DK).  QKV [n][ld]: [q: heads * DK | k: heads * DK |
+// grid (heads, ceil(dv / COLS)), 4 * COLS threads (COLS = 64, or 32 where that fills more SMs), dynamic shared memory lightning_chunk_smem<DK, COLS>.  QKV [n][ld]: [q: heads * DK | k: heads * DK |
 // v: heads * dv] behind the activation; dv a multiple of 8, ld a multiple of 8.  A CTA walks the chunk's tokens LC_TOKENS at a time (next tile in flight by
-// cp.async) for LC_COLS columns of one head's state.  Warp w: read-out of token rows 16 (w & 3) .. for 32 of the columns; state columns
-// (rows of the transpose) 16 (w & 3) .. for half of the DK entries, as accumulator fragments of the update product.
+// cp.async) for COLS columns of one head's state.  Warp w: read-out of token rows 16 (w & 3) .. for 32 of the columns; state columns (rows of the
+// transpose) 16 (w mod COLS / 16) .. for half of the DK entries, as accumulator fragments of the update product.
 // ---------------------------------------------------------------------------------------------------------------------
 #define LC_TOKENS 64
-#define LC_COLS 64
-#define LC_THREADS 256
-template <int DK> __host__ __device__ constexpr size_t lightning_chunk_smem() { // Q, K x 2 buffers, V x 2, split decayed V, split S^T
-    return (size_t)2 * (4 * LC_TOKENS * (DK + 8) + 2 * LC_TOKENS * (LC_COLS + 8) + 2 * LC_TOKENS * (LC_COLS + 8) + 2 * LC_COLS * (DK + 8));
+template <int DK, int COLS> __host__ __device__ constexpr size_t lightning_chunk_smem() { // Q, K x 2 buffers, V x 2, split decayed V, split S^T
+    return (size_t)2 * (4 * LC_TOKENS * (DK + 8) + 2 * LC_TOKENS * (COLS + 8) + 2 * LC_TOKENS * (COLS + 8) + 2 * COLS * (DK + 8));
 }
 __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const void *row) {
     const unsigned a = (unsigned)__cvta_generic_to_shared(row);
@@ -161,11 +159,11 @@ __device__ __forceinline__ void split_bf16(float x, float y, unsigned &hi, unsig
     lo = pack_bf16(x - bf_lo(hi), y - bf_hi(hi));
 }
 
-template <int DK>
-__global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__restrict__ QKV, int ld, LightningArgs a, float *__restrict__ S, int n, const StepState *__restrict__ st,
+template <int DK, int COLS>
+__global__ void __launch_bounds__(4 * COLS) k_lightning_chunk(const bf16 *__restrict__ QKV, int ld, LightningArgs a, float *__restrict__ S, int n, const StepState *__restrict__ st,
                                                                 float *__restrict__ Y, int ldy) {
     extern __shared__ __align__(16) unsigned char lsm[];
-    constexpr int T = LC_TOKENS, QW = DK + 8, VW = LC_COLS + 8;
+    constexpr int T = LC_TOKENS, QW = DK + 8, VW = COLS + 8, LC_THREADS = 4 * COLS, LC_COLS = COLS;
     typedef bf16 QRow[QW];
     typedef bf16 VRow[VW];
     QRow *Qs = reinterpret_cast<QRow *>(lsm), *Ks = Qs + 2 * T; // [buffer * T + token]
@@ -173,7 +171,8 @@ __global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__re
     VRow *Vs = reinterpret_cast<VRow *>(SL + LC_COLS), *VH = Vs + 2 * T, *VL = VH + T;
     __shared__ float pw[T + 1]; // powers of the head's decay
     const int h = blockIdx.x, j0 = blockIdx.y * LC_COLS, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int rb = (warp & 3) * 16, half = warp >> 2;
+    const int rb = (warp & 3) * 16, half = warp >> 2;                           // read-out: token rows, block of 32 columns
+    const int sb = warp % (COLS / 16) * 16, shalf = warp / (COLS / 16);         // state: columns, half of the DK entries
     const int qo = h * DK, ko = a.heads * DK + h * DK, vo = 2 * a.heads * DK + h * a.dv + j0;
     auto fetch = [&](int t0, int buf) {
         const int nt = n - t0 < T ? n - t0 : T;
@@ -192,11 +191,11 @@ __global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__re
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(0, 0);
-    if (tid <= T) pw[tid] = powf(a.decay[h], (float)tid);
-    // S^T rows j0 + rb + g (+ 8), entries half * DK / 2 + i * 8 + 2 t (+ 1)
+    for (int i = tid; i <= T; i += LC_THREADS) pw[i] = powf(a.decay[h], (float)i);
+    // S^T rows j0 + sb + g (+ 8), entries shalf * DK / 2 + i * 8 + 2 t (+ 1)
     float s[DK / 16][4];
-    float *Sg = S + ((size_t)h * a.dv + j0 + rb + g) * DK + half * (DK / 2) + 2 * t;
-    const bool in0 = j0 + rb + g < a.dv, in1 = j0 + rb + g + 8 < a.dv, fresh = st->pos == 0;
+    float *Sg = S + ((size_t)h * a.dv + j0 + sb + g) * DK + shalf * (DK / 2) + 2 * t;
+    const bool in0 = j0 + sb + g < a.dv, in1 = j0 + sb + g + 8 < a.dv, fresh = st->pos == 0;
 #pragma unroll
     for (int i = 0; i < DK / 16; i++) {
         const float2 z = make_float2(0.0f, 0.0f);
@@ -214,11 +213,11 @@ __global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__re
 #pragma unroll
         for (int i = 0; i < DK / 16; i++) {
             unsigned hi, lo;
-            const int c = half * (DK / 2) + i * 8 + 2 * t;
+            const int c = shalf * (DK / 2) + i * 8 + 2 * t;
             split_bf16(s[i][0], s[i][1], hi, lo);
-            *reinterpret_cast<unsigned *>(&SH[rb + g][c]) = hi; *reinterpret_cast<unsigned *>(&SL[rb + g][c]) = lo;
+            *reinterpret_cast<unsigned *>(&SH[sb + g][c]) = hi; *reinterpret_cast<unsigned *>(&SL[sb + g][c]) = lo;
             split_bf16(s[i][2], s[i][3], hi, lo);
-            *reinterpret_cast<unsigned *>(&SH[rb + g + 8][c]) = hi; *reinterpret_cast<unsigned *>(&SL[rb + g + 8][c]) = lo;
+            *reinterpret_cast<unsigned *>(&SH[sb + g + 8][c]) = hi; *reinterpret_cast<unsigned *>(&SL[sb + g + 8][c]) = lo;
         }
         for (int e = tid; e < T * (LC_COLS / 2); e += LC_THREADS) {
             const int r = e / (LC_COLS / 2), c = (e % (LC_COLS / 2)) * 2;
@@ -303,13 +302,13 @@ __global__ void __launch_bounds__(LC_THREADS) k_lightning_chunk(const bf16 *__re
 #pragma unroll
         for (int kk = 0; kk < T / 16; kk++) {
             unsigned vh[4], vl[4];
-            const int r = kk * 16 + (lane >> 4) * 8 + (lane & 7), c = rb + ((lane >> 3) & 1) * 8; // four 8 x 8 blocks, transposed: [value][token]
+            const int r = kk * 16 + (lane >> 4) * 8 + (lane & 7), c = sb + ((lane >> 3) & 1) * 8; // four 8 x 8 blocks, transposed: [value][token]
             ldmatrix_x4_trans(vh, &VH[r][c]);
             ldmatrix_x4_trans(vl, &VL[r][c]);
 #pragma unroll
             for (int i = 0; i < DK / 16; i++) {
                 unsigned b[2];
-                ldmatrix_x2_trans(b, &K[kk * 16 + (lane & 15)][half * (DK / 2) + i * 8]);
+                ldmatrix_x2_trans(b, &K[kk * 16 + (lane & 15)][shalf * (DK / 2) + i * 8]);
                 mma_bf16_16816(s[i], vh, b);
                 mma_bf16_16816(s[i], vl, b);
             }

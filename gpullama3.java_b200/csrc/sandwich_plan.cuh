@@ -229,11 +229,17 @@ static int ly_enqueue_lightning(b200_plan *p, bool decode, int n, const StepStat
     if (h16 && L.chunkwise && n >= LC_CHUNK_MIN) {
         const int w = 2 * L.qd + L.vd;
         if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, P, Y.maxP, w, (int)ly::ACT_SILU, Y.LQ16, w, ly::TokenGate{}))) return rc;
-        const dim3 cgrid(s.heads, (s.value_dim + LC_COLS - 1) / LC_COLS);
+        const bool wide = s.heads * ((s.value_dim + 63) / 64) >= p->n_sms;
+        const int cols = wide ? 64 : 32;
+        const dim3 cgrid(s.heads, (s.value_dim + cols - 1) / cols), cblock(4 * cols);
         const ly::bf16 *qkv = Y.LQ16;
-        if (s.key_dim == 32) rc = launch_k(p, false, ly::k_lightning_chunk<32>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<32>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
-        else if (s.key_dim == 64) rc = launch_k(p, false, ly::k_lightning_chunk<64>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<64>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
-        else rc = launch_k(p, false, ly::k_lightning_chunk<128>, cgrid, dim3(LC_THREADS), ly::lightning_chunk_smem<128>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
+#define LY_CHUNK_CASE(DK) \
+        if (s.key_dim == DK) rc = wide ? launch_k(p, false, ly::k_lightning_chunk<DK, 64>, cgrid, cblock, ly::lightning_chunk_smem<DK, 64>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO) \
+                                       : launch_k(p, false, ly::k_lightning_chunk<DK, 32>, cgrid, cblock, ly::lightning_chunk_smem<DK, 32>(), qkv, w, a, R.S, n, st, Y.DO, Y.maxDO);
+        LY_CHUNK_CASE(32)
+        LY_CHUNK_CASE(64)
+        LY_CHUNK_CASE(128)
+#undef LY_CHUNK_CASE
         ++*nl;
     } else switch (ly::lightning_reg_rows(s.key_dim)) {
     case 1: rc = launch_k(p, false, ly::k_lightning_scan<1>, grid, block, (size_t)0, P, Y.maxP, a, R.S, n, st, Y.DO, Y.maxDO); break;
