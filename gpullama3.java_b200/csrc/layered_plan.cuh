@@ -179,9 +179,9 @@ struct Layered {
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
     // per-layer token input: second embedding table [vocab][layers * side_dim], gated rows
     ly::bf16 *side_emb = nullptr, *SIDE16 = nullptr;
-    float *SIDE32 = nullptr;
+    float *SIDE32 = nullptr, *SIDEF = nullptr; // SIDEF: FP32 result of the gate product on the tcgen05 route [cap][side_pad]
     int side_pad = 0;
-    CUtensorMap m_side;
+    CUtensorMap m_side, m_sidef_c;
 };
 
 // What ly_project needs to take the tcgen05 route: operand and result descriptors (nullptr = CUDA-core / mma.sync kernels).
@@ -739,10 +739,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
         if (s.window > Y.max_window) Y.max_window = s.window;
         if (s.value_dim > Y.max_att_dv) Y.max_att_dv = s.value_dim;
     }
-    if (c.side_dim > 0) { // gate rows in whole tcgen05 tiles; their FP32 result takes the projection buffer
-        Y.side_pad = (c.side_dim + 127) / 128 * 128;
-        if (Y.side_pad > Y.maxP) Y.maxP = Y.side_pad;
-    }
+    Y.side_pad = (c.side_dim + 127) / 128 * 128; // gate rows of the per-layer token input in whole tcgen05 tiles
     {
         int maxK = E > Y.maxO ? E : Y.maxO;
         if (Y.maxD > maxK) maxK = Y.maxD; // reduction width of W_x
@@ -779,8 +776,14 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
             CK(set_max_dyn(ly::k_window_attention_mma<256, 128>, Y.smem_max));
             CK(set_max_dyn(ly::k_window_attention_mma<256, 128, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_delta_prep, Y.smem_max));
-            CK(set_max_dyn(ly::k_selective_scan<32, 16>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 1>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 2>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 4>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 8>, Y.smem_max));
             CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 16>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<SEL_LANES, 32>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<32, 8>, Y.smem_max));
+            CK(set_max_dyn(ly::k_selective_scan<32, 16>, Y.smem_max));
             CK(set_max_dyn(ly::k_lightning_chunk<32, 32>, Y.smem_max));
             CK(set_max_dyn(ly::k_lightning_chunk<32, 64>, Y.smem_max));
             CK(set_max_dyn(ly::k_lightning_chunk<64, 32>, Y.smem_max));
@@ -1045,7 +1048,7 @@ static int ly_build(b200_plan *p, const b200_layered_config *cfg, const b200_lay
     }
     if (c.side_dim > 0) {
         if ((rc = dalloc(p, &Y.SIDE32, rows32 * c.side_dim * 4))) return rc;
-        if (!Y.f32 && (rc = dalloc(p, &Y.SIDE16, cap * c.side_dim * 2))) return rc;
+        if (!Y.f32 && ((rc = dalloc(p, &Y.SIDE16, cap * c.side_dim * 2)) || (rc = dalloc(p, &Y.SIDEF, cap * Y.side_pad * 4)))) return rc;
     }
     if ((rc = dalloc(p, &Y.Y, cap * E * 4))) return rc;
     if ((rc = dalloc(p, &Y.PROJ, cap * Y.maxP * 4))) return rc;

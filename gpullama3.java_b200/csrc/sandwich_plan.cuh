@@ -198,7 +198,7 @@ static void ly_sandwich_tc_init(b200_plan *p) {
     auto fits = [](int N, int K) { return N % 128 == 0 && K % 64 == 0; };
     const bool xp_c = Y.XP && Y.maxX % 4 == 0 && pg::make_map_c(&Y.m_xp_c, Y.XP, rows, Y.maxX) == 0;
     const bool dt_c = Y.Q && Y.maxQ % 4 == 0 && pg::make_map_c(&Y.m_dt_c, Y.Q, rows, Y.maxQ) == 0;
-    const bool side_a = D > 0 && D % 64 == 0 && Y.maxP % 4 == 0 && pg::make_map(&Y.m_side, Y.SIDE16, rows, D, pg::BM) == 0;
+    const bool side_a = D > 0 && D % 64 == 0 && pg::make_map(&Y.m_side, Y.SIDE16, rows, D, pg::BM) == 0 && pg::make_map_c(&Y.m_sidef_c, Y.SIDEF, rows, Y.side_pad) == 0;
     for (LyLayer &L : Y.layers) {
         const b200_layer_spec &s = L.s;
         if (s.mixer == B200_MIXER_ATTENTION_SCAN) {
@@ -298,7 +298,7 @@ static int ly_enqueue_selective(b200_plan *p, bool decode, int n, const StepStat
     const int z_off = L.x_off + I;
     a.vec = I % 4 == 0 && N % 4 == 0 && Rk % 4 == 0 && z_off % 4 == 0 && Y.maxP % 4 == 0 && Y.maxX % 4 == 0 && Y.maxQ % 4 == 0 && Y.maxD % 4 == 0;
     const int lpc = ly::sel_lanes(N), ch = SEL_THREADS / lpc;
-    const dim3 grid((I + ch - 1) / ch), block(SEL_THREADS);
+    const dim3 grid((I + ch - 1) / ch), block(SEL_BLOCK);
     const float *U = Y.DLT, *PX = Y.XP, *DT = Y.Q, *Z = Y.PROJ + z_off;
     float *o32 = h16 ? nullptr : Y.ATT32 + L.ad;
     ly::bf16 *o16 = h16 ? Y.ATT16 + L.ad : nullptr;
@@ -312,7 +312,8 @@ static int ly_enqueue_selective(b200_plan *p, bool decode, int n, const StepStat
     case 2: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 2>, grid, block, ly::sel_smem(SEL_LANES, 2), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
     case 4: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 4>, grid, block, ly::sel_smem(SEL_LANES, 4), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
     case 8: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 8>, grid, block, ly::sel_smem(SEL_LANES, 8), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
-    default: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 16>, grid, block, ly::sel_smem(SEL_LANES, 16), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    case 16: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 16>, grid, block, ly::sel_smem(SEL_LANES, 16), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
+    default: return launch_k(p, false, ly::k_selective_scan<SEL_LANES, 32>, grid, block, ly::sel_smem(SEL_LANES, 32), U, Y.maxD, PX, Y.maxX, DT, Y.maxQ, Z, Y.maxP, a, R.S, n, st, o32, o16, L.gd);
     }
 }
 
@@ -359,9 +360,9 @@ static int ly_enqueue_side(b200_plan *p, bool decode, int n, const StepState *st
     *nl += 2;
     if (h16 && Y.tc && L.tc_side) {
         LyTc t, t2;
-        t.a = &Y.m_a; t.b = &L.m_tsg; t.c = &Y.m_proj_c;
-        if ((rc = ly_project<ly::EPI_STORE>(p, false, n, nullptr, Y.A16, L.w_sgate, nullptr, Y.side_pad, E, Y.PROJ, nullptr, Y.maxP, 0, &t))) return rc;
-        if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, (const float *)Y.PROJ, Y.maxP, D, (int)ly::ACT_GELU_TANH, Y.SIDE16, D, tg))) return rc;
+        t.a = &Y.m_a; t.b = &L.m_tsg; t.c = &Y.m_sidef_c;
+        if ((rc = ly_project<ly::EPI_STORE>(p, false, n, nullptr, Y.A16, L.w_sgate, nullptr, Y.side_pad, E, Y.SIDEF, nullptr, Y.side_pad, 0, &t))) return rc;
+        if ((rc = launch_k(p, false, ly::k_act_rows, dim3(n), dim3(256), (size_t)0, (const float *)Y.SIDEF, Y.side_pad, D, (int)ly::ACT_GELU_TANH, Y.SIDE16, D, tg))) return rc;
         t2.a = &Y.m_side; t2.b = &L.m_tsp; t2.c = &Y.m_y_c;
         ++*nl;
         return ly_project<ly::EPI_STORE>(p, false, n, nullptr, Y.SIDE16, L.w_sproj, nullptr, E, D, Y.Y, nullptr, E, 0, &t2);
