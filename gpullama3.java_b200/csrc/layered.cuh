@@ -1142,14 +1142,19 @@ __global__ void __launch_bounds__(BM * 2) k_window_attention_mma(const float *__
         const float *gate = (a.gate_src ? a.gate_src + (size_t)r * a.gate_ld : P + (size_t)r * ldp) + (a.gate_off >= 0 ? a.gate_off : qd + kd + vd) +
                             (a.gate_heads ? (size_t)h : (size_t)h * DV);
         const float ghead = a.gate && a.gate_heads ? 1.0f / (1.0f + expf(-gate[0])) : 1.0f;
+        const bool entries = a.gate && !a.gate_heads;
+        float2 gv[DV / 8]; // a gate per output entry: the row's loads are in flight together
+        if (entries) {
+#pragma unroll
+            for (int j = 0; j < DV / 8; j++) gv[j] = __ldg(reinterpret_cast<const float2 *>(gate + j * 8 + 2 * t));
+        }
 #pragma unroll
         for (int j = 0; j < DV / 8; j++) {
             const int d = j * 8 + 2 * t;
             float v0 = o[j][2 * rr] * inv * ghead, v1 = o[j][2 * rr + 1] * inv * ghead;
-            if (a.gate && !a.gate_heads) {
-                const float2 gv = *reinterpret_cast<const float2 *>(gate + d);
-                v0 *= sigmoid_fast(gv.x);
-                v1 *= sigmoid_fast(gv.y);
+            if (entries) {
+                v0 *= sigmoid_fast(gv[j].x);
+                v1 *= sigmoid_fast(gv[j].y);
             }
             if (out32) *reinterpret_cast<float2 *>(out32 + (size_t)r * ldo + (size_t)h * DV + d) = make_float2(v0, v1); // FP32 results (what a later subtraction reads)
             else *reinterpret_cast<unsigned *>(out + (size_t)r * ldo + (size_t)h * DV + d) = pack_bf16(v0, v1);

@@ -56,14 +56,15 @@ __global__ void __launch_bounds__(LIGHT_THREADS) k_lightning_scan(const float *_
             pv = t < nt && j0 + i < a.dv ? P[(size_t)(t0 + t) * ldp + vo + i] : 0.0f;
         }
     };
-    auto store = [&](int buf) { // silu(0) = 0: rows and tokens beyond the end stay zero
+    auto store = [&](int buf, int nt) { // silu(0) = 0: rows beyond dk stay zero; nothing reads a token beyond the end
 #pragma unroll
         for (int k = 0; k < LB; k++) {
             const int e = tid + k * LIGHT_THREADS;
+            if (e / RW >= nt) continue;
             (&ks[buf][0][0])[e] = siluf_(pk[k]);
             (&qs[buf][0][0])[e] = siluf_(pq[k]);
         }
-        if (tid < TB * LIGHT_COLS) (&vs[buf][0][0])[tid] = siluf_(pv);
+        if (tid < TB * LIGHT_COLS && tid / LIGHT_COLS < nt) (&vs[buf][0][0])[tid] = siluf_(pv);
     };
     load(0);
     float *Sg = S + ((size_t)h * a.dv + (column ? col : 0)) * RW;
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(LIGHT_THREADS) k_lightning_scan(const float *_
         for (int i = 0; i < R; i++) s[i] = 0.0f;
     }
     const float dec = a.decay[h];
-    store(0);
+    store(0, n < TB ? n : TB);
     __syncthreads();
     int buf = 0;
     for (int t0 = 0; t0 < n; t0 += TB, buf ^= 1) {
@@ -126,7 +127,7 @@ __global__ void __launch_bounds__(LIGHT_THREADS) k_lightning_scan(const float *_
             acc += __shfl_xor_sync(0xffffffffu, acc, 1);
             if (slice == 0 && column) Y[(size_t)(t0 + t) * ldy + (size_t)h * a.dv + col] = acc;
         }
-        if (more) store(buf ^ 1); // that buffer was consumed before the barrier that started this iteration
+        if (more) store(buf ^ 1, n - t0 - TB < TB ? n - t0 - TB : TB); // that buffer was consumed before the barrier that started this iteration
         __syncthreads();
     }
     if (!column) return;

@@ -257,6 +257,7 @@ struct ConvArgs {
     const float *bias_out; // [C] (nullable)
     int silu;              // 1: SiLU on the result
 };
+#define LY_CONV_FEW 4  // convolutions of at most this many taps keep their inputs in registers
 #define LY_CONV_ROWS 4 // consecutive rows of a channel per thread: their loads are independent and in flight together
 __global__ void __launch_bounds__(256) k_conv_rows(const float *__restrict__ P, int ldp, int c_off, ConvArgs a, float *__restrict__ cstate, float *__restrict__ out32, int ldo,
                                                    bf16 *__restrict__ out16, int ldo16, const StepState *__restrict__ st, int n) {
@@ -266,20 +267,37 @@ __global__ void __launch_bounds__(256) k_conv_rows(const float *__restrict__ P, 
     float acc[LY_CONV_ROWS];
 #pragma unroll
     for (int i = 0; i < LY_CONV_ROWS; i++) acc[i] = bo;
-    for (int m = 0; m < a.taps; m++) {
-        const int back = a.taps - 1 - m;
-        const float wm = a.w[(size_t)c * a.taps + m];
+    const int pos0 = st->pos;
+    if (a.taps <= LY_CONV_FEW) { // every input of the four rows once, all of them and the weights in flight before the first is used
+        float x[LY_CONV_ROWS + LY_CONV_FEW - 1], w[LY_CONV_FEW];
 #pragma unroll
-        for (int i = 0; i < LY_CONV_ROWS; i++) {
-            const int r = r0 + i, pos = st->pos + r;
-            if (r >= n || pos - back < 0) continue;
-            const float x = back <= r ? P[(size_t)(r - back) * ldp + c_off + c] + bi : cstate[(size_t)((pos - back) % a.cring) * a.C + c];
-            acc[i] = fmaf(wm, x, acc[i]);
+        for (int k = 0; k < LY_CONV_FEW; k++) w[k] = k < a.taps ? a.w[(size_t)c * a.taps + a.taps - 1 - k] : 0.0f; // w[k]: the tap k tokens back
+#pragma unroll
+        for (int k = 0; k < LY_CONV_ROWS + LY_CONV_FEW - 1; k++) { // input of row r0 + k - (LY_CONV_FEW - 1)
+            const int r = r0 + k - (LY_CONV_FEW - 1);
+            const bool used = k >= LY_CONV_FEW - a.taps && r < n && pos0 + r >= 0;
+            x[k] = !used ? 0.0f : r >= 0 ? P[(size_t)r * ldp + c_off + c] + bi : cstate[(size_t)((pos0 + r) % a.cring) * a.C + c];
+        }
+#pragma unroll
+        for (int k = LY_CONV_FEW - 1; k >= 0; k--)
+#pragma unroll
+            for (int i = 0; i < LY_CONV_ROWS; i++) acc[i] = fmaf(w[k], x[i + LY_CONV_FEW - 1 - k], acc[i]);
+    } else {
+        for (int m = 0; m < a.taps; m++) {
+            const int back = a.taps - 1 - m;
+            const float wm = a.w[(size_t)c * a.taps + m];
+#pragma unroll
+            for (int i = 0; i < LY_CONV_ROWS; i++) {
+                const int r = r0 + i, pos = pos0 + r;
+                if (r >= n || pos - back < 0) continue;
+                const float x = back <= r ? P[(size_t)(r - back) * ldp + c_off + c] + bi : cstate[(size_t)((pos - back) % a.cring) * a.C + c];
+                acc[i] = fmaf(wm, x, acc[i]);
+            }
         }
     }
 #pragma unroll
     for (int i = 0; i < LY_CONV_ROWS; i++) {
-        const int r = r0 + i, pos = st->pos + r;
+        const int r = r0 + i, pos = pos0 + r;
         if (r >= n) break;
         // a later launch reads at most taps - 1 rows back
         if (r + a.taps > n) cstate[(size_t)(pos % a.cring) * a.C + c] = P[(size_t)r * ldp + c_off + c] + bi;
