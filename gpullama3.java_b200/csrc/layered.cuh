@@ -774,9 +774,10 @@ __global__ void __launch_bounds__(NTH) k_qk_prep(float *__restrict__ P, int ldp,
 // One CTA per (row, head): scores of the window into shared memory, softmax with the sink term, weighted value sum, gate.
 // Scores: a group of dk/4 lanes (at most a warp) owns a key and reads its row with coalesced 128-bit loads; values: a group of
 // dv/4 threads owns every groups-th key.  Sizes that are no multiple of 4 take scalar loads.
-// gridDim.z > 1 splits the window of a (row, head) over several CTAs; the last one to arrive merges the parts.
+// gridDim.z > 1 splits the window of a (row, head) over up to that many CTAs; the last one to arrive merges the parts.
 // Dynamic shared memory: att_smem_floats(dk, window) floats.
 #define LY_ATT_THREADS 256
+#define LY_ATT_SPLIT_KEYS 32
 // Scratch of a launch that splits every (row, head) over gridDim.z CTAs (the decode step: one row, few heads, many SMs):
 // per part the unnormalised weighted value sum o[dv] and {maximum, sum of exponentials}; count = arrival counter per (row, head).
 struct KeySplit {
@@ -793,7 +794,7 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
     __shared__ float red[32];
     __shared__ int s_last;
     const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int splits = gridDim.z, z = blockIdx.z;
+    const int z = blockIdx.z;
     const int qd = a.heads * a.dk, kd = a.kv_heads * a.dk, vd = a.kv_heads * a.dv;
     const int g = h / (a.heads / a.kv_heads);
     const int gk = a.maps > 1 ? g * a.maps + h % a.maps : a.k_heads > 0 ? h / (a.heads / a.k_heads) : g;
@@ -801,6 +802,9 @@ __global__ void __launch_bounds__(LY_ATT_THREADS) k_window_attention(const float
     const int pos = st->pos + r;
     int lo = window_first(a, pos);
     int nk = pos - lo + 1;
+    // as many of the launch's splits as have LY_ATT_SPLIT_KEYS keys to work on (every CTA of a (row, head) counts the same number)
+    const int want = (nk + LY_ATT_SPLIT_KEYS - 1) / LY_ATT_SPLIT_KEYS, splits = want < (int)gridDim.z ? want : (int)gridDim.z;
+    if (z >= splits) return;
     if (splits > 1) { // this CTA's share of the window; everything below indexes keys as lo + j, j < nk
         const int chunk = (nk + splits - 1) / splits, jb = z * chunk;
         lo += jb;
