@@ -6,8 +6,10 @@
 //                       N(v; w) = v / sqrt(mean(v^2) + eps) * (w_off + w); also the embedding gather (x = scale * E[token], optionally
 //                       normalised); with post_plain the sublayer output is added as x += y * w_post (a layer scale behind a pre-norm);
 //                       the sublayer output may be a mixture of experts, assembled here from the chosen experts' rows and their weights;
+//   * k_norm_rows_reg   the same with the row in registers, for the shapes and steps that allow it;
 //   * k_matvec_bf16     decode projection: BF16 weight rows streamed with 128-bit loads, FP32 activation and accumulator,
 //                       bias or gated-activation epilogue (gelu_tanh(g) * u);
+//   * k_matvec_row_bf16 the same for matrices of few rows: a CTA per row;
 //   * k_gemm_f32 / k_gemm_bf16   prefill projections for any M, N, K: true FP32 on the CUDA cores, or BF16 operands on the
 //                       tensor cores (mma.sync m16n8k16, FP32 accumulation), same epilogues;
 //   * k_qk_prep         whole-projection RMS norm of q and of k (one statistic over ALL heads), optional rotation, K / V rows into the window ring;
